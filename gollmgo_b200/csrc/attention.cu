@@ -24,7 +24,7 @@
 
 template <typename TA, int DMAX>
 __device__ __forceinline__ void attn_tile(const AttnArgs& a, int nrows, const TA* const* qptr_s,
-                                          const int* pos_s, const int* head_s, int kvh, const int* bt, int lo_main,
+                                          const int* pos_s, const int* head_s, const float* scale_s, int kvh, const int* bt, int lo_main,
                                           int hi_main, int first_hi, float* smem, float* acc) {
   constexpr int NACC = ATT_BQ * DMAX / ATT_THREADS;
   const int d = a.d, dv = a.dv > 0 ? a.dv : a.d, ps = a.page_size;
@@ -90,8 +90,9 @@ __device__ __forceinline__ void attn_tile(const AttnArgs& a, int nrows, const TA
         const int p = pos_s[r];
         const bool ok = tok >= lo && tok < hi && tok <= p && (a.window <= 0 || tok > p - a.window || tok < a.keep_first) &&
                         (a.chunk <= 0 || tok >= (p / a.chunk) * a.chunk);
-        float sc = s[i] * a.scale;
+        float sc = s[i] * scale_s[r];
         if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
+        if (ok && a.slopes) sc -= a.slopes[head_s[r]] * (float)(p - tok);
         if (ok && a.dist_bias) sc += a.dist_bias[(size_t)a.dist_bucket[min(p - tok, a.dist_max)] * a.nh + head_s[r]];
         if (ok && a.head_bias) sc += a.head_bias[head_s[r]];
         Ss[r * ATT_BK + j] = ok ? sc : -INFINITY;
@@ -160,6 +161,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_prefill_kernel(AttnArgs a) {
   __shared__ const TA* qptr_s[ATT_BQ];
   __shared__ int pos_s[ATT_BQ];
   __shared__ int head_s[ATT_BQ];
+  __shared__ float scale_s[ATT_BQ];
   pdl_wait();
   const int b = a.tile_seq[blockIdx.x], q0 = a.tile_q0[blockIdx.x];
   const int h = blockIdx.y, kvh = h / (a.nh / a.nkv);
@@ -172,13 +174,14 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_prefill_kernel(AttnArgs a) {
     qptr_s[r] = r < nrows ? (const TA*)a.q + (size_t)(t0 + q0 + r) * a.q_stride + (size_t)h * a.d : nullptr;
     pos_s[r] = r < nrows ? qstart + q0 + r : -1;
     head_s[r] = h;
+    scale_s[r] = a.scale * query_temperature(a, qstart + q0 + r);
   }
   __syncthreads();
   const int first = qstart + q0, last = first + nrows - 1;
   int lo = a.window > 0 ? max(0, first - a.window + 1) : 0;
   if (a.chunk > 0) lo = max(lo, (first / a.chunk) * a.chunk);       // the chunk of the tile's first row starts earliest
   float acc[NACC];
-  attn_tile<TA, DMAX>(a, nrows, qptr_s, pos_s, head_s, kvh, a.block_tables + (size_t)b * a.bt_stride, lo, last + 1,
+  attn_tile<TA, DMAX>(a, nrows, qptr_s, pos_s, head_s, scale_s, kvh, a.block_tables + (size_t)b * a.bt_stride, lo, last + 1,
                       min(a.keep_first, lo), smem, acc);
   pdl_trigger();
   float* m_s = const_cast<float*>(attn_tile_max(a, smem));
@@ -225,6 +228,7 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_decode_kernel(AttnArgs a) {
   __shared__ const TA* qptr_s[ATT_BQ];
   __shared__ int pos_s[ATT_BQ];
   __shared__ int head_s[ATT_BQ];
+  __shared__ float scale_s[ATT_BQ];
   pdl_wait();
   const int G = a.nh / a.nkv, gchunks = (G + ATT_BQ - 1) / ATT_BQ;
   const int b = a.dec_seqs[blockIdx.x];
@@ -244,12 +248,13 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_decode_kernel(AttnArgs a) {
     qptr_s[r] = r < nrows ? (const TA*)a.q + (size_t)t * a.q_stride + (size_t)(kvh * G + g0 + r) * a.d : nullptr;
     pos_s[r] = r < nrows ? ctx - 1 : -1;
     head_s[r] = kvh * G + g0 + (r < nrows ? r : 0);
+    scale_s[r] = a.scale * query_temperature(a, max(ctx - 1, 0));
   }
   __syncthreads();
   float acc[NACC];
   if (lo < hi) {
     // the first slice also takes the first tokens that stay visible behind the window
-    attn_tile<TA, DMAX>(a, nrows, qptr_s, pos_s, head_s, kvh, a.block_tables + (size_t)b * a.bt_stride, lo, hi,
+    attn_tile<TA, DMAX>(a, nrows, qptr_s, pos_s, head_s, scale_s, kvh, a.block_tables + (size_t)b * a.bt_stride, lo, hi,
                         split == 0 ? min(a.keep_first, lo0) : 0, smem, acc);
   } else {
 #pragma unroll
@@ -541,7 +546,7 @@ extern "C" int gg_attn_prefill_x(const void* q, long long q_stride, const void* 
                                  void* out, int out_f32, int nh, int nkv, int d, int dv, int v_share,
                                  int page_size, int window, float scale, float softcap, int keep_first, int weights,
                                  const float* head_bias, const float* dist_bias, const int* dist_bucket, int dist_max, int chunk, const float* sink,
-                                 cudaStream_t stream) {
+                                 const float* slopes, float temp_coef, float temp_every, cudaStream_t stream) {
   AttnArgs a = {};
   a.q = q; a.q_stride = q_stride; a.kcache = kcache; a.vcache = vcache;
   a.block_tables = block_tables; a.bt_stride = bt_stride; a.cu_q_lens = cu_q_lens;
@@ -552,11 +557,12 @@ extern "C" int gg_attn_prefill_x(const void* q, long long q_stride, const void* 
   a.keep_first = window > 0 ? keep_first : 0; a.weights = weights; a.head_bias = head_bias;
   a.dist_bias = dist_bias; a.dist_bucket = dist_bucket; a.dist_max = dist_max;
   a.chunk = chunk > 0 ? chunk : 0; a.sink = sink;
+  a.slopes = slopes; a.temp_coef = temp_coef; a.temp_every = temp_every;
   int rc = check_common(a, "attn_prefill_x");
   if (rc) return rc;
   GG_REQUIRE(weights == 0 || weights == 1, "attn_prefill_x: unknown kind of weights %d", weights);
   GG_REQUIRE(!dist_bias || (dist_bucket && dist_max >= 0), "attn_prefill_x: a distance bias needs its bucket table");
-  GG_REQUIRE(!(weights && (a.chunk || sink)), "attn_prefill_x: chunks and a sink go with softmax weights");
+  GG_REQUIRE(!(weights && (a.chunk || sink || slopes || temp_every > 0.f)), "attn_prefill_x: chunks, a sink, slopes and a query temperature go with softmax weights");
   // what the mma.sync kernels compute: softmax without these extras, or sigmoid weights with all of them
   const bool plain = (!a.keep_first && !weights && !head_bias && !dist_bias) || attn_mma_x_sigmoid_supported(a);
   if (a.chunk || a.sink) allow_mma = allow_mma && attn_mma_x_chunk_sink_supported();
@@ -575,7 +581,7 @@ extern "C" int gg_attn_decode_x(const void* q, long long q_stride, const void* k
                                 int dv, int v_share, int page_size, int window, float scale, float softcap,
                                 int allow_mma, int keep_first, int weights, const float* head_bias,
                                 const float* dist_bias, const int* dist_bucket, int dist_max, int chunk, const float* sink,
-                                cudaStream_t stream) {
+                                const float* slopes, float temp_coef, float temp_every, cudaStream_t stream) {
   AttnArgs a = {};
   a.q = q; a.q_stride = q_stride; a.kcache = kcache; a.vcache = vcache;
   a.block_tables = block_tables; a.bt_stride = bt_stride; a.cu_q_lens = cu_q_lens;
@@ -586,11 +592,12 @@ extern "C" int gg_attn_decode_x(const void* q, long long q_stride, const void* k
   a.keep_first = window > 0 ? keep_first : 0; a.weights = weights; a.head_bias = head_bias;
   a.dist_bias = dist_bias; a.dist_bucket = dist_bucket; a.dist_max = dist_max;
   a.chunk = chunk > 0 ? chunk : 0; a.sink = sink;
+  a.slopes = slopes; a.temp_coef = temp_coef; a.temp_every = temp_every;
   int rc = check_common(a, "attn_decode_x");
   if (rc) return rc;
   GG_REQUIRE(weights == 0 || weights == 1, "attn_decode_x: unknown kind of weights %d", weights);
   GG_REQUIRE(!dist_bias || (dist_bucket && dist_max >= 0), "attn_decode_x: a distance bias needs its bucket table");
-  GG_REQUIRE(!(weights && (a.chunk || sink)), "attn_decode_x: chunks and a sink go with softmax weights");
+  GG_REQUIRE(!(weights && (a.chunk || sink || slopes || temp_every > 0.f)), "attn_decode_x: chunks, a sink, slopes and a query temperature go with softmax weights");
   if ((a.keep_first || weights || head_bias || dist_bias) && !attn_mma_x_sigmoid_supported(a))
     allow_mma = 0;                                                            // only the general kernel has these with softmax
   if (a.chunk) allow_mma = allow_mma && attn_mma_x_chunk_sink_supported();     // (the sink is the merge kernel's)

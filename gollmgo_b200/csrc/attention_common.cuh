@@ -43,7 +43,16 @@ struct AttnArgs {
   int chunk;                // > 0: the sequence is cut into chunks of this many positions, counted from 0, and a query sees
                             // only the keys of its own chunk (all kernels but the tcgen05 ones and the plain mma.sync ones)
   const float* sink;        // [nh] or null: exp(sink[h]) is one more term of the softmax denominator, with no key and no value
+  const float* slopes;      // [nh] or null: slopes[h] * (i - j) is taken off the scaled score (softmax weights)
+  float temp_coef;          // the query at position p is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
+  float temp_every;         // (0: it is not; softmax weights).  Applied to the score's scale, so q is not rounded once more
 };
+
+// the factor on the query at position p (1 where the layer has none)
+__device__ __forceinline__ float query_temperature(const AttnArgs& a, int p) {
+  if (!(a.temp_every > 0.f)) return 1.f;
+  return 1.f + a.temp_coef * logf(floorf(__fdiv_rn((float)(p + 1), a.temp_every)) + 1.f);
+}
 
 // General kernels (attention.cu)
 int attn_prefill_general(const AttnArgs& a, int dtype, int num_tiles, cudaStream_t stream);
@@ -61,7 +70,7 @@ int attn_prefill_mma_x(const AttnArgs& a, int num_tiles, cudaStream_t stream);  
 // a.weights == 1 (sigmoid weights, kept first keys, biases by head and distance) on the same kernels
 #define ATTN_MMA_X_MAX_DIST 16384      // entries of the distance table that fit in shared memory beside the tiles
 bool attn_mma_x_sigmoid_supported(const AttnArgs& a);
-// a.chunk and a.sink with softmax weights on the same kernels
+// a.chunk, a.sink, a.slopes and the query temperature with softmax weights on the same kernels
 bool attn_mma_x_chunk_sink_supported();
 int attn_decode_mma_x(const AttnArgs& a, int n_dec, cudaStream_t stream);        // partial results; the caller merges
 // large batches: the tiles of all (token, kv head) pairs cut into equal ranges, one per CTA

@@ -1124,6 +1124,9 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_prefill_mma_x_kernel(AttnArg
   // chunked: the first key each of this thread's two rows sees, and the first any row of the warp sees
   const int cs0 = a.chunk > 0 ? (max(pos0, 0) / a.chunk) * a.chunk : 0, cs1 = a.chunk > 0 ? (max(pos1, 0) / a.chunk) * a.chunk : 0;
   const int wfirst = a.chunk > 0 ? ((first + wrow0) / a.chunk) * a.chunk : 0;
+  // this head's slope over the distance (base-2 exponents) and the two rows' scales (a query temperature is part of them)
+  const float slope = !SIG && a.slopes ? a.slopes[h] * LOG2E : 0.f;
+  const float scale0 = SIG ? a.scale : a.scale * query_temperature(a, pos0), scale1 = SIG ? a.scale : a.scale * query_temperature(a, pos1);
 
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[DV / 8][4];
@@ -1183,7 +1186,15 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_prefill_mma_x_kernel(AttnArg
             const int pos = (e & 2) ? pos1 : pos0;
             const bool ok = ((e & 2) ? row1_ok : row0_ok) && tk >= lo && tk <= pos &&
                             (a.window <= 0 || tk > pos - a.window) && tk >= ((e & 2) ? cs1 : cs0);
-            s[j][e] = ok ? score_exp2(s[j][e], scale, cap, inv_cap) : -INFINITY;
+            s[j][e] = ok ? score_exp2(s[j][e], (e & 2) ? scale1 : scale0, cap, inv_cap) : -INFINITY;
+          }
+        }
+        if (slope != 0.f) {                        // (a masked score stays -inf)
+          const float away0 = (float)(pos0 - kb - c2), away1 = (float)(pos1 - kb - c2);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[j][e] -= slope * (((e & 2) ? away1 : away0) - (float)(j * 8 + (e & 1)));
           }
         }
         softmax_update<DV, 8>(s, m, l, o, p);
@@ -1269,7 +1280,10 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_decode_mma_x_kernel(AttnArgs
     unsigned qf[DK / 16][4];
     const __nv_bfloat16* qbase = (const __nv_bfloat16*)a.q + (size_t)t * a.q_stride + (size_t)head0 * DK;
     load_q_frags<DK>(qf, [&](int r) { return r < nrows ? qbase + (size_t)r * DK : nullptr; });
-    const float scale = a.scale, cap = a.softcap, inv_cap = cap > 0.f ? 1.f / cap : 0.f;
+    // rows g and g + 8 of the tile are heads head0 + g and head0 + g + 8 (clamped where the group is smaller)
+    const float slope0 = !SIG && a.slopes ? a.slopes[head0 + min(g, nrows - 1)] * LOG2E : 0.f;
+    const float slope1 = !SIG && a.slopes ? a.slopes[head0 + min(g + 8, nrows - 1)] * LOG2E : 0.f;
+    const float scale = SIG ? a.scale : a.scale * query_temperature(a, ctx - 1), cap = a.softcap, inv_cap = cap > 0.f ? 1.f / cap : 0.f;
     for (int it = 0; it < ntiles; ++it) {
       if (it + 1 < ntiles) {
         const int st = (it + 1) % STAGES;
@@ -1341,6 +1355,11 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_decode_mma_x_kernel(AttnArgs
             s[j][2] = tk < hi ? score_exp2(s[j][2], scale, cap, inv_cap) : -INFINITY;
             s[j][1] = tk + 1 < hi ? score_exp2(s[j][1], scale, cap, inv_cap) : -INFINITY;
             s[j][3] = tk + 1 < hi ? score_exp2(s[j][3], scale, cap, inv_cap) : -INFINITY;
+            if (a.slopes) {
+              const float away = (float)(ctx - 1 - tk);
+              s[j][0] -= slope0 * away; s[j][2] -= slope1 * away;
+              s[j][1] -= slope0 * (away - 1.f); s[j][3] -= slope1 * (away - 1.f);
+            }
           }
           softmax_update<DV, 2>(s, m, l, o, p);
         }

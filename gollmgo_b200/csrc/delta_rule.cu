@@ -377,7 +377,7 @@ delta_recur_kernel(const float* __restrict__ qkv, const float* __restrict__ beta
 }
 
 // ---------------------------------------------------------------- the gated norm of the result
-// grid (T, H): out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate[t, h, :])
+// grid (T, H): out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate[t, h, :]); w null: no weight
 template <typename TA>
 __global__ void delta_out_kernel(const float* __restrict__ o_raw, const TA* __restrict__ gate, long long gate_stride,
                                  const float* __restrict__ w, float eps, int H, int dv, int gate_act, TA* __restrict__ out) {
@@ -393,7 +393,7 @@ __global__ void delta_out_kernel(const float* __restrict__ o_raw, const TA* __re
   TA* y = out + (size_t)t * H * dv + (size_t)h * dv;
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
     const float z = to_f32(gr[c]);
-    y[c] = from_f32<TA>(o[c] * f * w[c] * (gate_act == 1 ? 1.f / (1.f + expf(-z)) : silu_f(z)));
+    y[c] = from_f32<TA>(o[c] * f * (w ? w[c] : 1.f) * (gate_act == 1 ? 1.f / (1.f + expf(-z)) : silu_f(z)));
   }
 }
 

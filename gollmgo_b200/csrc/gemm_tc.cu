@@ -41,7 +41,8 @@ template <int MODE>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                void* __restrict__ out, int M, int N, int K, int tiles_m, int num_tiles,
-               int* __restrict__ status, int withhold_loads, const int* __restrict__ tile_group, int group_rows) {
+               int* __restrict__ status, int withhold_loads, const int* __restrict__ tile_group, int group_rows,
+               const int* __restrict__ row_entry, const float* __restrict__ row_scale) {
   constexpr int BN = 256;
   constexpr unsigned A_BYTES = TC_BM * TC_BK * 2, B_BYTES = BN * TC_BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
   extern __shared__ unsigned char tc_smem_raw[];
@@ -146,6 +147,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
       const int buf = local & 1;
       const int m0 = (t % tiles_m) * TC_BM, n0 = (t / tiles_m) * n_out_tile;
       const int row = m0 + quarter * 32 + lane;
+      float rs = 1.f;                            // grouped product: a factor on the row, from the list of what the rows hold
+      if (MODE == TC_OUT_SILU && row_scale && row < M) {
+        const int entry = row_entry[row];
+        if (entry >= 0) rs = row_scale[entry];
+      }
       if (!mbar_wait(acc_full0 + 8 * buf, (local >> 1) & 1)) { atomicExch(status, TC_ERR_ACC_WAIT); atomicExch(&abort_s, 1); break; }
       if (*(volatile int*)&abort_s) break;
       tc_fence_after();
@@ -160,8 +166,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           float v[32];
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
-            const float gj = __uint_as_float(g[j]);
-            v[j] = gj / (1.f + __expf(-gj)) * __uint_as_float(u[j]);
+            const float gj = __uint_as_float(g[j]) * rs;
+            v[j] = gj / (1.f + __expf(-gj)) * (__uint_as_float(u[j]) * rs);
           }
           if (row < M) store_row32(o + c, v, N - (n0 + c));
         }
@@ -228,7 +234,8 @@ int gg_make_map_2d(CUtensorMap* map, const void* ptr, int rows, int cols, long l
 // left untouched unless a wait inside the kernel ran out (then non-zero).
 static int gemm_tc_launch(const void* x, long long ldx, const void* W, void* out, int M, int N, int K,
                           int mode, int* status, int withhold_loads, cudaStream_t stream,
-                          const int* tile_group = nullptr, int groups = 1);
+                          const int* tile_group = nullptr, int groups = 1, const int* row_entry = nullptr,
+                          const float* row_scale = nullptr);
 
 extern "C" int gg_gemm_tc(const void* x, long long ldx, const void* W, void* out, int M, int N, int K,
                           int mode, int* status, cudaStream_t stream) {
@@ -239,13 +246,17 @@ extern "C" int gg_gemm_tc(const void* x, long long ldx, const void* W, void* out
 // [groups, 2N, K] gated), and every block of 128 rows of x belongs to one of them:
 // tile_group[i] (device memory, written by a kernel earlier in the stream) is the group of rows
 // 128 i .. 128 i + 127, or < 0 for a block that belongs to none and is skipped.  The rows of a
-// group therefore start at a multiple of 128 (the caller pads).  M = rows of x and out.
+// group therefore start at a multiple of 128 (the caller pads).  M = rows of x and out.  row_scale (gated
+// only): the products of row r are multiplied by row_scale[row_entry[r]] before the activation, where
+// row_entry[r] >= 0.
 extern "C" int gg_gemm_tc_grouped(const void* x, long long ldx, const void* W, void* out, int M, int N, int K,
-                                  int mode, const int* tile_group, int groups, int* status, cudaStream_t stream) {
+                                  int mode, const int* tile_group, int groups, const int* row_entry,
+                                  const float* row_scale, int* status, cudaStream_t stream) {
   GG_REQUIRE(tile_group != nullptr && groups > 0, "gemm_tc_grouped: no groups given");
   GG_REQUIRE(M % TC_BM == 0, "gemm_tc_grouped: %d rows are no multiple of %d", M, TC_BM);
   GG_REQUIRE(mode == TC_OUT_BF16 || mode == TC_OUT_SILU, "gemm_tc_grouped: mode %d", mode);
-  return gemm_tc_launch(x, ldx, W, out, M, N, K, mode, status, 0, stream, tile_group, groups);
+  GG_REQUIRE(!row_scale || (row_entry && mode == TC_OUT_SILU), "gemm_tc_grouped: factors on rows go with the gated product and a row list");
+  return gemm_tc_launch(x, ldx, W, out, M, N, K, mode, status, 0, stream, tile_group, groups, row_entry, row_scale);
 }
 
 // Self-test of the bounded waits: the same launch, but the loads are withheld, so no barrier a
@@ -258,7 +269,7 @@ extern "C" int gg_gemm_tc_withheld(const void* x, long long ldx, const void* W, 
 
 static int gemm_tc_launch(const void* x, long long ldx, const void* W, void* out, int M, int N, int K,
                           int mode, int* status, int withhold_loads, cudaStream_t stream,
-                          const int* tile_group, int groups) {
+                          const int* tile_group, int groups, const int* row_entry, const float* row_scale) {
   GG_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_tc: bad sizes M=%d N=%d K=%d", M, N, K);
   GG_REQUIRE(K % 8 == 0 && ldx % 8 == 0, "gemm_tc: K=%d and the row stride %lld of x must be multiples of 8", K, ldx);
   GG_REQUIRE(((size_t)x % 16) == 0 && ((size_t)W % 16) == 0, "gemm_tc: x and W must be 16-byte aligned");
@@ -297,7 +308,7 @@ static int gemm_tc_launch(const void* x, long long ldx, const void* W, void* out
       if (e != cudaSuccess) return gg_fail(GG_ERR_CUDA, "gemm_tc: %s", cudaGetErrorString(e));            \
       set = true;                                                                                         \
     }                                                                                                     \
-    e = gg_launch(gemm_tc_kernel<MODE>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, out, M, N, K, tiles_m, num_tiles, status, withhold_loads, tile_group, w_rows); \
+    e = gg_launch(gemm_tc_kernel<MODE>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, out, M, N, K, tiles_m, num_tiles, status, withhold_loads, tile_group, w_rows, row_entry, row_scale); \
   } while (0)
   if (mode == TC_OUT_BF16) TC_LAUNCH(TC_OUT_BF16);
   else if (mode == TC_OUT_F32) TC_LAUNCH(TC_OUT_F32);

@@ -9,7 +9,9 @@
 //   W_g:              [N, K] row-major ([2N, K] if gated: gate rows, then up rows) at W + g * rows * K
 //   out row r, columns [g * o_group_cols, g * o_group_cols + Np): the N results, then zeros
 //   epilogue:         gated: silu(x Wg^T) * (x Wu^T);   gate given: the row is multiplied by
-//                     sigmoid(gate[A row, gate_col0 + g])   (an output gate per head)
+//                     sigmoid(gate[A row, gate_col0 + g])   (an output gate per head);
+//                     row_scale given: row r's products are multiplied by row_scale[row_index ? row_index[r] : r]
+//                     before the activation (a factor on the input row, without rounding the row again)
 //
 // No host code learns how many rows a group has: the grid is sized for the worst case and a CTA
 // whose tile lies past its group's rows returns.  A row's result depends on that row and on W_g
@@ -40,6 +42,7 @@ struct GroupedArgs {
   const int* offsets;
   int M, G, N, K, Np, gated;
   const void* gate; long long ldg; int gate_col0;
+  const float* row_scale;
 };
 
 template <typename TA> struct GgmZero;
@@ -63,6 +66,7 @@ __global__ void __launch_bounds__(GGM_THREADS, (sizeof(TA) == 2 ? (GATED ? 2 : 4
   constexpr int C_BYTES = NB * GGM_BM * GGM_LDC * (int)sizeof(float);
   __shared__ __align__(32) unsigned char raw[AB_BYTES > C_BYTES ? AB_BYTES : C_BYTES];
   __shared__ int arow_s[GGM_BM];
+  __shared__ float scale_s[GGM_BM];
   TA* As = reinterpret_cast<TA*>(raw);
   TA* Bs = As + GGM_BM * LD;                                    // [NB][GGM_BN * LD]
   float* Cs = reinterpret_cast<float*>(raw);                    // [NB][GGM_BM * GGM_LDC], over the tiles once they are used up
@@ -85,7 +89,11 @@ __global__ void __launch_bounds__(GGM_THREADS, (sizeof(TA) == 2 ? (GATED ? 2 : 4
   }
   const int n0 = blockIdx.x * GGM_BN;
   const int nrows = min(GGM_BM, r_end - r0);
-  if (tid < GGM_BM) arow_s[tid] = tid < nrows ? (a.row_index ? a.row_index[r0 + tid] / a.row_div : r0 + tid) : -1;
+  if (tid < GGM_BM) {
+    const int entry = tid < nrows ? (a.row_index ? a.row_index[r0 + tid] : r0 + tid) : -1;
+    arow_s[tid] = entry < 0 ? -1 : (a.row_index ? entry / a.row_div : entry);
+    scale_s[tid] = entry >= 0 && a.row_scale ? a.row_scale[entry] : 1.f;
+  }
   __syncthreads();
   const int N = a.N, K = a.K;
   const TA* A = (const TA*)a.A + (size_t)g * a.a_group_cols;
@@ -201,9 +209,9 @@ __global__ void __launch_bounds__(GGM_THREADS, (sizeof(TA) == 2 ? (GATED ? 2 : 4
     if (r >= nrows || col >= a.Np) continue;
     float v = 0.f;
     if (col < N) {
-      v = Cs[r * GGM_LDC + c];
+      v = Cs[r * GGM_LDC + c] * scale_s[r];
       if (GATED) {
-        const float u = Cs1[r * GGM_LDC + c];
+        const float u = Cs1[r * GGM_LDC + c] * scale_s[r];
         v = v / (1.f + expf(-v)) * u;
       }
       if (a.gate) {
@@ -233,6 +241,7 @@ __global__ void __launch_bounds__(GGM_THREADS, 2) grouped_gemm_ring_kernel(Group
   constexpr int STAGE_ELEMS = A_ELEMS + NB * B_ELEMS;
   extern __shared__ __align__(128) unsigned char ring_raw[];
   __shared__ int arow_s[GGM_BM];
+  __shared__ float scale_s[GGM_BM];
   TA* stages = reinterpret_cast<TA*>(ring_raw);
   float* Cs = reinterpret_cast<float*>(ring_raw);                // over the ring once it has drained
   pdl_trigger();
@@ -254,7 +263,11 @@ __global__ void __launch_bounds__(GGM_THREADS, 2) grouped_gemm_ring_kernel(Group
   }
   const int n0 = blockIdx.x * GGM_BN;
   const int nrows = min(GGM_BM, r_end - r0);
-  if (tid < GGM_BM) arow_s[tid] = tid < nrows ? (a.row_index ? a.row_index[r0 + tid] / a.row_div : r0 + tid) : -1;
+  if (tid < GGM_BM) {
+    const int entry = tid < nrows ? (a.row_index ? a.row_index[r0 + tid] : r0 + tid) : -1;
+    arow_s[tid] = entry < 0 ? -1 : (a.row_index ? entry / a.row_div : entry);
+    scale_s[tid] = entry >= 0 && a.row_scale ? a.row_scale[entry] : 1.f;
+  }
   __syncthreads();
   const int N = a.N, K = a.K;
   const TA* A = (const TA*)a.A + (size_t)g * a.a_group_cols;
@@ -333,9 +346,9 @@ __global__ void __launch_bounds__(GGM_THREADS, 2) grouped_gemm_ring_kernel(Group
     if (r >= nrows || col >= a.Np) continue;
     float v = 0.f;
     if (col < N) {
-      v = Cs[r * GGM_LDC + c];
+      v = Cs[r * GGM_LDC + c] * scale_s[r];
       if (GATED) {
-        const float u = Cs1[r * GGM_LDC + c];
+        const float u = Cs1[r * GGM_LDC + c] * scale_s[r];
         v = v / (1.f + expf(-v)) * u;
       }
       if (a.gate) {
@@ -350,7 +363,7 @@ __global__ void __launch_bounds__(GGM_THREADS, 2) grouped_gemm_ring_kernel(Group
 extern "C" int gg_grouped_gemm(const void* A, long long lda, long long a_group_cols, const int* row_index,
                                int row_div, const void* W, void* out, long long ldo, long long o_group_cols,
                                const int* offsets, int M, int G, int N, int K, int Np, int gated,
-                               const void* gate, long long ldg, int gate_col0, int act_dtype,
+                               const void* gate, long long ldg, int gate_col0, const float* row_scale, int act_dtype,
                                cudaStream_t stream) {
   GG_REQUIRE(M >= 0 && G > 0 && N > 0 && K > 0 && Np >= N, "grouped_gemm: bad sizes M=%d G=%d N=%d K=%d Np=%d", M, G, N, K, Np);
   GG_REQUIRE(A && W && out, "grouped_gemm: a pointer is null");
@@ -360,7 +373,7 @@ extern "C" int gg_grouped_gemm(const void* A, long long lda, long long a_group_c
   a.A = A; a.lda = lda; a.a_group_cols = a_group_cols; a.row_index = row_index; a.row_div = row_div;
   a.W = W; a.out = out; a.ldo = ldo; a.o_group_cols = o_group_cols; a.offsets = offsets;
   a.M = M; a.G = G; a.N = N; a.K = K; a.Np = Np; a.gated = gated;
-  a.gate = gate; a.ldg = ldg; a.gate_col0 = gate_col0;
+  a.gate = gate; a.ldg = ldg; a.gate_col0 = gate_col0; a.row_scale = row_scale;
   const int row_tiles = offsets ? (M + GGM_BM - 1) / GGM_BM + G : (M + GGM_BM - 1) / GGM_BM;
   GG_REQUIRE(row_tiles <= 65535 && G <= 65535, "grouped_gemm: %d row tiles or %d groups are too many for one launch", row_tiles, G);
   dim3 grid((Np + GGM_BN - 1) / GGM_BN, row_tiles, offsets ? 1 : G);

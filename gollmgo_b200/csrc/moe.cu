@@ -3,12 +3,14 @@
 //
 // gg_moe_route:   z[t, e] = h[t] . Wr[e] + b[e] in float32; the `top` largest logits of a token
 //                 (ties: the lower index) are its experts, weights = softmax over those alone, or
-//                 the softmax over all experts renormalised over the chosen; optionally only
-//                 experts of the best groups can be chosen (moe_pick)
+//                 the softmax over all experts renormalised over the chosen, or each chosen logit's
+//                 sigmoid as it is; optionally only experts of the best groups can be chosen (moe_pick);
+//                 optionally one more row of Wr, whose product with h[t] is left in gate[t] (the logit of a
+//                 shared expert's gate)
 // gg_moe_align:   the (token, choice) pairs sorted by expert: offsets[e] .. offsets[e+1] are the
 //                 places of expert e in `sorted` (values t * top + j), `place` is the inverse
-// gg_moe_combine: out[t] = sum_j weight[t, j] * y[place[t * top + j]] (+ shared[t]), float32 sums
-//                 in the order of j
+// gg_moe_combine: out[t] = sum_j weight[t, j] * y[place[t * top + j]] (+ shared[t], times the sigmoid
+//                 of its gate where there is one), float32 sums in the order of j; no weights: plain sum
 // The products between them are gg_grouped_gemm's (grouped_gemm.cu).
 #include "common.cuh"
 
@@ -35,7 +37,8 @@ __device__ __forceinline__ void route_load(const __nv_bfloat16* w, float (&v)[8]
 
 // One warp picks a token's experts from its logits zr[E] (shared memory, overwritten) and weighs them.
 // weigh = 0: weights = softmax over the chosen logits alone.  weigh = 1: scores = softmax over all
-// experts, weights = the chosen scores divided by their sum (+ 1e-20).  groups > 1: the experts form
+// experts, weights = the chosen scores divided by their sum (+ 1e-20).  weigh = 2: weights = the sigmoid
+// of each chosen logit, not normalised (the largest sigmoids are the largest logits').  groups > 1: the experts form
 // that many equal groups of neighbours, a group's score is its best expert's, and only experts of the
 // `keep` best groups can be chosen.  Ties: the lower index.
 __device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, int groups, int keep, int lane,
@@ -102,6 +105,8 @@ __device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, i
       float sum = 0.f;
       for (int j = 0; j < top; ++j) { val[j] = expf(val[j] - zmax) / zsum; sum += val[j]; }
       for (int j = 0; j < top; ++j) wgt[j] = val[j] / (sum + 1e-20f);
+    } else if (weigh == 2) {
+      for (int j = 0; j < top; ++j) wgt[j] = 1.f / (1.f + expf(-val[j]));
     } else {
       const float m = val[0];                        // the largest comes first
       float sum = 0.f;
@@ -114,7 +119,7 @@ __device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, i
 template <typename TA, int TOK>
 __global__ void moe_route_kernel(const TA* __restrict__ h, const TA* __restrict__ wr, const float* __restrict__ bias,
                                  int T, int D, int E, int top, int weigh, int groups, int keep,
-                                 int* __restrict__ idx, float* __restrict__ wgt, int vec) {
+                                 int* __restrict__ idx, float* __restrict__ wgt, float* __restrict__ gate, int vec) {
   __shared__ float z[TOK][MOE_MAX_EXPERTS];
   extern __shared__ __align__(16) float xs[];              // TOK rows of D floats
   constexpr int VPT = 16 / (int)sizeof(TA);
@@ -127,7 +132,8 @@ __global__ void moe_route_kernel(const TA* __restrict__ h, const TA* __restrict_
     xs[e] = r < nt ? to_f32(h[(size_t)(t0 + r) * D + (e - r * D)]) : 0.f;
   }
   __syncthreads();
-  for (int e = warp; e < E; e += nw) {
+  const int rows = E + (gate ? 1 : 0);
+  for (int e = warp; e < rows; e += nw) {
     const TA* w = wr + (size_t)e * D;
     float s[TOK];
 #pragma unroll
@@ -156,7 +162,10 @@ __global__ void moe_route_kernel(const TA* __restrict__ h, const TA* __restrict_
 #pragma unroll
     for (int r = 0; r < TOK; ++r) {
       const float tot = warp_sum(s[r]);
-      if (lane == 0) z[r][e] = tot + (bias ? bias[e] : 0.f);
+      if (lane == 0) {
+        if (e < E) z[r][e] = tot + (bias ? bias[e] : 0.f);
+        else if (r < nt) gate[t0 + r] = tot;
+      }
     }
   }
   __syncthreads();
@@ -166,7 +175,7 @@ __global__ void moe_route_kernel(const TA* __restrict__ h, const TA* __restrict_
 
 // The choice alone, from logits a product has already made (long steps: z = h Wr^T in float32 by the
 // vendor library from the bfloat16 rows): one warp a token adds the bias, picks and weighs.
-__global__ void moe_topk_kernel(const float* __restrict__ z, const float* __restrict__ bias, int T, int E, int top,
+__global__ void moe_topk_kernel(const float* __restrict__ z, long long z_stride, const float* __restrict__ bias, int T, int E, int top,
                                 int weigh, int groups, int keep, int* __restrict__ idx, float* __restrict__ wgt) {
   extern __shared__ float zs[];                            // warps x E
   pdl_trigger();
@@ -175,7 +184,7 @@ __global__ void moe_topk_kernel(const float* __restrict__ z, const float* __rest
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= T) return;
   float* zr = zs + warp * E;
-  for (int e = lane; e < E; e += 32) zr[e] = z[(size_t)t * E + e] + (bias ? bias[e] : 0.f);
+  for (int e = lane; e < E; e += 32) zr[e] = z[t * z_stride + e] + (bias ? bias[e] : 0.f);
   __syncwarp();
   moe_pick(zr, E, top, weigh, groups, keep, lane, idx + (size_t)t * top, wgt + (size_t)t * top);
 }
@@ -249,22 +258,25 @@ __global__ void moe_gather_kernel(const TA* __restrict__ x, const int* __restric
 
 template <typename TA>
 __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restrict__ place, const float* __restrict__ wgt,
-                                   const TA* __restrict__ shared_out, TA* __restrict__ out, int D, int top) {
+                                   const TA* __restrict__ shared_out, const float* __restrict__ gate, long long gate_stride,
+                                   TA* __restrict__ out, int D, int top) {
   pdl_trigger();
   pdl_wait();
   const size_t t = blockIdx.x;
+  const float sg = gate ? 1.f / (1.f + expf(-gate[t * gate_stride])) : 1.f;      // on the shared expert
   if (D % 4 == 0) {                              // rows of every buffer are then 8-byte aligned at least
     for (int c = threadIdx.x * 4; c < D; c += blockDim.x * 4) {
       float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
       for (int j = 0; j < top; ++j) {
-        const float w = wgt[t * top + j];
+        const float w = wgt ? wgt[t * top + j] : 1.f;
         const TA* r = y + (size_t)place[t * top + j] * D + c;
         s0 = fmaf(w, to_f32(r[0]), s0); s1 = fmaf(w, to_f32(r[1]), s1);
         s2 = fmaf(w, to_f32(r[2]), s2); s3 = fmaf(w, to_f32(r[3]), s3);
       }
       if (shared_out) {
         const TA* r = shared_out + t * D + c;
-        s0 += to_f32(r[0]); s1 += to_f32(r[1]); s2 += to_f32(r[2]); s3 += to_f32(r[3]);
+        s0 = fmaf(sg, to_f32(r[0]), s0); s1 = fmaf(sg, to_f32(r[1]), s1);
+        s2 = fmaf(sg, to_f32(r[2]), s2); s3 = fmaf(sg, to_f32(r[3]), s3);
       }
       TA* o = out + t * D + c;
       o[0] = from_f32<TA>(s0); o[1] = from_f32<TA>(s1); o[2] = from_f32<TA>(s2); o[3] = from_f32<TA>(s3);
@@ -274,21 +286,22 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restri
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     float s = 0.f;
     for (int j = 0; j < top; ++j)
-      s = fmaf(wgt[t * top + j], to_f32(y[(size_t)place[t * top + j] * D + c]), s);
-    if (shared_out) s += to_f32(shared_out[t * D + c]);
+      s = fmaf(wgt ? wgt[t * top + j] : 1.f, to_f32(y[(size_t)place[t * top + j] * D + c]), s);
+    if (shared_out) s = fmaf(sg, to_f32(shared_out[t * D + c]), s);
     out[t * D + c] = from_f32<TA>(s);
   }
 }
 
 static int check_pick(const char* who, int E, int top, int weigh, int groups, int keep) {
-  GG_REQUIRE(weigh == 0 || weigh == 1, "%s: unknown way %d of weighing the chosen experts", who, weigh);
+  GG_REQUIRE(weigh >= 0 && weigh <= 2, "%s: unknown way %d of weighing the chosen experts", who, weigh);
   GG_REQUIRE(groups >= 1 && keep >= 1 && keep <= groups && E % groups == 0, "%s: %d experts in %d groups of which %d are kept", who, E, groups, keep);
   GG_REQUIRE(top <= keep * (E / groups), "%s: %d choices from %d groups of %d experts", who, top, keep, E / groups);
   return GG_OK;
 }
 
 extern "C" int gg_moe_route(const void* h, const void* wr, const float* bias, int T, int D, int E, int top,
-                            int weigh, int groups, int keep, int* idx, float* wgt, int act_dtype, cudaStream_t stream) {
+                            int weigh, int groups, int keep, int* idx, float* wgt, float* gate, int act_dtype,
+                            cudaStream_t stream) {
   GG_REQUIRE(T >= 0 && D > 0 && E > 0 && top > 0 && top <= E, "moe_route: bad sizes T=%d D=%d E=%d top=%d", T, D, E, top);
   GG_REQUIRE(E <= MOE_MAX_EXPERTS && top <= MOE_MAX_TOP, "moe_route: at most %d experts and %d choices a token (got %d, %d)",
              MOE_MAX_EXPERTS, MOE_MAX_TOP, E, top);
@@ -304,7 +317,7 @@ extern "C" int gg_moe_route(const void* h, const void* wr, const float* bias, in
 #define ROUTE_LAUNCH(T_, N_)                                                                                     \
   do {                                                                                                           \
     if (smem > 28 * 1024) cudaFuncSetAttribute(moe_route_kernel<T_, N_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-    gg_launch(moe_route_kernel<T_, N_>, dim3(blocks), dim3(threads), smem, stream, (const T_*)h, (const T_*)wr, bias, T, D, E, top, weigh, groups, keep, idx, wgt, vec); \
+    gg_launch(moe_route_kernel<T_, N_>, dim3(blocks), dim3(threads), smem, stream, (const T_*)h, (const T_*)wr, bias, T, D, E, top, weigh, groups, keep, idx, wgt, gate, vec); \
   } while (0)
   if (act_dtype == GG_F32) {
     if (tok == 1) ROUTE_LAUNCH(float, 1); else ROUTE_LAUNCH(float, ROUTE_TOK);
@@ -315,16 +328,16 @@ extern "C" int gg_moe_route(const void* h, const void* wr, const float* bias, in
   return gg_check_launch("moe_route");
 }
 
-extern "C" int gg_moe_topk(const float* z, const float* bias, int T, int E, int top, int weigh, int groups, int keep,
+extern "C" int gg_moe_topk(const float* z, long long z_stride, const float* bias, int T, int E, int top, int weigh, int groups, int keep,
                            int* idx, float* wgt, cudaStream_t stream) {
   GG_REQUIRE(T >= 0 && E > 0 && top > 0 && top <= E && E <= MOE_MAX_EXPERTS && top <= MOE_MAX_TOP,
              "moe_topk: bad sizes T=%d E=%d top=%d", T, E, top);
-  GG_REQUIRE(z && idx && wgt, "moe_topk: a pointer is null");
+  GG_REQUIRE(z && idx && wgt && z_stride >= E, "moe_topk: a pointer is null or the rows are too short");
   if (int rc = check_pick("moe_topk", E, top, weigh, groups, keep)) return rc;
   if (T == 0) return GG_OK;
   const int warps = 4;
   gg_launch(moe_topk_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), (size_t)warps * E * sizeof(float), stream,
-            z, bias, T, E, top, weigh, groups, keep, idx, wgt);
+            z, z_stride, bias, T, E, top, weigh, groups, keep, idx, wgt);
   return gg_check_launch("moe_topk");
 }
 
@@ -355,18 +368,18 @@ extern "C" int gg_moe_gather(const void* x, const int* sorted, int slots, int to
   return gg_check_launch("moe_gather");
 }
 
-extern "C" int gg_moe_combine(const void* y, const int* place, const float* wgt, const void* shared_out, void* out,
-                              int T, int D, int top, int act_dtype, cudaStream_t stream) {
+extern "C" int gg_moe_combine(const void* y, const int* place, const float* wgt, const void* shared_out,
+                              const float* gate, long long gate_stride, void* out, int T, int D, int top, int act_dtype, cudaStream_t stream) {
   GG_REQUIRE(T >= 0 && D > 0 && top > 0, "moe_combine: bad sizes T=%d D=%d top=%d", T, D, top);
-  GG_REQUIRE(y && place && wgt && out, "moe_combine: a pointer is null");
+  GG_REQUIRE(y && place && out && (shared_out || !gate), "moe_combine: a pointer is null");
   if (T == 0) return GG_OK;
   const int threads = D >= 1024 ? 256 : 128;
   if (act_dtype == GG_F32)
     gg_launch(moe_combine_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)y, place, wgt, (const float*)shared_out,
-              (float*)out, D, top);
+              gate, gate_stride, (float*)out, D, top);
   else if (act_dtype == GG_BF16)
     gg_launch(moe_combine_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, (const __nv_bfloat16*)y, place, wgt,
-              (const __nv_bfloat16*)shared_out, (__nv_bfloat16*)out, D, top);
+              (const __nv_bfloat16*)shared_out, gate, gate_stride, (__nv_bfloat16*)out, D, top);
   else
     return gg_fail(GG_ERR_INVALID, "moe_combine: unknown dtype %d", act_dtype);
   return gg_check_launch("moe_combine");

@@ -576,14 +576,18 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
                  a_group_cols: int = 0, o_group_cols: int = 0, n_padded: Optional[int] = None,
                  offsets: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None, row_div: int = 1,
                  rows: Optional[int] = None, gated: bool = False, gate: Optional[torch.Tensor] = None,
-                 gate_col0: int = 0) -> None:
+                 gate_col0: int = 0, row_scale: Optional[torch.Tensor] = None) -> None:
     """out_g = a_g @ w_g^T for every group g (csrc/grouped_gemm.cu).  w [groups, n (2n if gated), k].
     Without ``offsets`` every group has the first ``rows`` rows of a and reads columns
     g * a_group_cols .. + k of them; with ``offsets`` [groups + 1] group g has rows offsets[g] ..
     offsets[g + 1] of the row list (``rows`` = its length), row r reading row row_index[r] // row_div
     of a.  Results go to out[r, g * o_group_cols : + n_padded] (zeros past n).  ``gate``: row r of
-    group g is multiplied by sigmoid(gate[a row, gate_col0 + g])."""
-    _cuda(w, offsets, row_index)
+    group g is multiplied by sigmoid(gate[a row, gate_col0 + g]).  ``row_scale`` (float32): the products
+    of row r are multiplied by row_scale[row_index[r]] (row_scale[r] without a row list) before the
+    activation: a factor on the input row that does not round it again."""
+    _cuda(w, offsets, row_index, row_scale)
+    if row_scale is not None and row_scale.dtype != torch.float32:
+        raise KernelError("grouped_gemm: the factors on rows are float32")
     if a.dtype != w.dtype or out.dtype != a.dtype or a.stride(-1) != 1 or out.stride(-1) != 1:
         raise KernelError("grouped_gemm: a, w and out of one dtype, rows contiguous")
     if w.numel() != groups * (2 if gated else 1) * n * k:
@@ -593,7 +597,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
                                  int(row_div), _p(w), _p(out), ctypes.c_longlong(out.stride(0)),
                                  ctypes.c_longlong(o_group_cols), _p(offsets), M, groups, n, k,
                                  int(n_padded if n_padded is not None else n), int(gated), _p(gate),
-                                 ctypes.c_longlong(gate.stride(0) if gate is not None else 0), int(gate_col0),
+                                 ctypes.c_longlong(gate.stride(0) if gate is not None else 0), int(gate_col0), _p(row_scale),
                                  dtype_code(a.dtype), _stream()))
 
 
@@ -611,32 +615,37 @@ def head_gate(a: torch.Tensor, gates: torch.Tensor, col0: int, heads: int) -> No
 MOE_MAX_EXPERTS, MOE_MAX_TOP = 1024, 32
 
 
-MOE_WEIGH = {"softmax_chosen": 0, "softmax_all": 1}
+MOE_WEIGH = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2}
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], top: int,
-              idx: torch.Tensor, wgt: torch.Tensor, weigh: str = "softmax_chosen", groups: int = 1, keep: int = 1) -> None:
+              idx: torch.Tensor, wgt: torch.Tensor, weigh: str = "softmax_chosen", groups: int = 1, keep: int = 1,
+              gate: Optional[torch.Tensor] = None) -> None:
     """Float32 logits h @ w_router^T + bias; idx [T, top] int32 = the largest, wgt [T, top]
     float32 = softmax over those ("softmax_chosen"), or the softmax over all experts divided by the
-    chosen ones' sum ("softmax_all").  ``groups`` > 1: only experts of the ``keep`` groups (of
-    neighbouring experts) with the best expert can be chosen."""
-    _cuda(h, w_router, bias, idx, wgt)
+    chosen ones' sum ("softmax_all"), or each chosen logit's sigmoid as it is ("sigmoid").  ``groups`` > 1:
+    only experts of the ``keep`` groups (of neighbouring experts) with the best expert can be chosen.
+    ``gate`` (float32 [T]): w_router has one row more than there are experts, whose product with h goes there."""
+    _cuda(h, w_router, bias, idx, wgt, gate)
     T, D = h.shape
-    E = w_router.shape[0]
+    E = w_router.shape[0] - (1 if gate is not None else 0)
+    if gate is not None and (gate.dtype != torch.float32 or gate.numel() < T):
+        raise KernelError("moe_route: the gate's logits are float32 [T]")
     if w_router.dtype != h.dtype or w_router.shape[1] != D or idx.dtype != torch.int32 or wgt.dtype != torch.float32 \
             or (bias is not None and bias.dtype != torch.float32):
         raise KernelError("moe_route: router of the rows' dtype, bias and weights float32, choices int32")
     _check(lib().gg_moe_route(_p(h), _p(w_router), _p(bias), T, D, E, top, MOE_WEIGH[weigh], int(groups), int(keep),
-                               _p(idx), _p(wgt), dtype_code(h.dtype), _stream()))
+                               _p(idx), _p(wgt), _p(gate), dtype_code(h.dtype), _stream()))
 
 
 def moe_topk(z: torch.Tensor, bias: Optional[torch.Tensor], top: int, idx: torch.Tensor, wgt: torch.Tensor,
-             weigh: str = "softmax_chosen", groups: int = 1, keep: int = 1) -> None:
-    """moe_route's choice from logits z [T, E] (float32) that a product has already made."""
+             weigh: str = "softmax_chosen", groups: int = 1, keep: int = 1, experts: Optional[int] = None) -> None:
+    """moe_route's choice from logits z [T, E] (float32) that a product has already made (``experts``: only
+    that many of z's columns are experts)."""
     _cuda(z, bias, idx, wgt)
     if z.dtype != torch.float32 or idx.dtype != torch.int32 or wgt.dtype != torch.float32:
         raise KernelError("moe_topk: logits and weights float32, choices int32")
-    _check(lib().gg_moe_topk(_p(z), _p(bias), z.shape[0], z.shape[1], top, MOE_WEIGH[weigh], int(groups), int(keep),
+    _check(lib().gg_moe_topk(_p(z), ctypes.c_longlong(z.stride(0)), _p(bias), z.shape[0], int(experts or z.shape[1]), top, MOE_WEIGH[weigh], int(groups), int(keep),
                               _p(idx), _p(wgt), _stream()))
 
 
@@ -660,28 +669,36 @@ def moe_gather(x: torch.Tensor, order: torch.Tensor, top: int, out: torch.Tensor
 
 
 def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_group: torch.Tensor, groups: int,
-                    gated: bool = False) -> None:
+                    gated: bool = False, row_entry: Optional[torch.Tensor] = None,
+                    row_scale: Optional[torch.Tensor] = None) -> None:
     """The tcgen05 product (gemm_tc) over groups: rows 128 i .. of x belong to group tile_group[i]
     (< 0: to none, skipped) and are multiplied with that group's matrix w[g] ([groups, N, K]; gated:
-    [groups, 2N, K], out = silu(x Wg^T) * (x Wu^T)).  bfloat16; rows of x a multiple of 128."""
+    [groups, 2N, K], out = silu(x Wg^T) * (x Wu^T)).  bfloat16; rows of x a multiple of 128.  ``row_scale``
+    (gated, float32): the products of row r are multiplied by row_scale[row_entry[r]] before the activation."""
     global tc_launched
     M, K = x.shape
     N = out.shape[1]
     if w.numel() != groups * (2 if gated else 1) * N * K or out.shape[0] != M or not out.is_contiguous() \
             or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("gemm_tc_grouped: shapes or dtypes do not fit")
-    _cuda(w, out, tile_group)
+    _cuda(w, out, tile_group, row_entry, row_scale)
+    if row_scale is not None and (row_scale.dtype != torch.float32 or row_entry is None or row_entry.numel() < M):
+        raise KernelError("gemm_tc_grouped: float32 factors with a row list as long as x")
     tc_launched = True
     _check(lib().gg_gemm_tc_grouped(_p(x), ctypes.c_longlong(x.stride(0)), _p(w), _p(out), M, N, K, 2 if gated else 0,
-                                    _p(tile_group), groups, _p(tc_status(x.device)), _stream()))
+                                    _p(tile_group), groups, _p(row_entry), _p(row_scale), _p(tc_status(x.device)), _stream()))
 
 
-def moe_combine(y: torch.Tensor, place: torch.Tensor, wgt: torch.Tensor, shared: Optional[torch.Tensor],
-                out: torch.Tensor, top: int) -> None:
-    """out[t] = sum_j wgt[t, j] * y[place[t * top + j]] (+ shared[t])."""
+def moe_combine(y: torch.Tensor, place: torch.Tensor, wgt: Optional[torch.Tensor], shared: Optional[torch.Tensor],
+                out: torch.Tensor, top: int, gate: Optional[torch.Tensor] = None) -> None:
+    """out[t] = sum_j wgt[t, j] * y[place[t * top + j]] (+ shared[t]); wgt None: weights of 1; ``gate`` (float32
+    column view [T, 1] or [T]): the shared row is multiplied by sigmoid(gate[t])."""
+    if gate is not None and (gate.dtype != torch.float32 or gate.shape[0] != out.shape[0]):
+        raise KernelError("moe_combine: the gate's logits are float32, one a token")
     _cuda(y, place, wgt, shared, out)
     T, D = out.shape
-    _check(lib().gg_moe_combine(_p(y), _p(place), _p(wgt), _p(shared), _p(out), T, D, top, dtype_code(out.dtype), _stream()))
+    _check(lib().gg_moe_combine(_p(y), _p(place), _p(wgt), _p(shared), _p(gate),
+                                ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _p(out), T, D, top, dtype_code(out.dtype), _stream()))
 
 
 # ---------------------------------------------------------------- attention of any make (general kernels)
@@ -722,7 +739,8 @@ def attn_prefill_x(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcache:
                    num_tiles64: int = 0, allow_mma: bool = True, keep_first: int = 0, sigmoid_weights: bool = False,
                    head_bias: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
                    dist_bucket: Optional[torch.Tensor] = None, chunk: int = 0,
-                   sink: Optional[torch.Tensor] = None) -> None:
+                   sink: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
+                   temperature=None) -> None:
     """Causal attention of prompt portions with keys of size d, values of size dv, ``v_share`` key
     heads to a value head, optional window and capped scores; out [T, nh*dv] in the cache's type or
     float32.  ``tile_*`` list tiles of 16 queries (general kernel, float32 arithmetic), ``tile64_*``
@@ -733,8 +751,10 @@ def attn_prefill_x(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcache:
     With softmax these three are the general kernel's alone; with sigmoid weights the mma.sync kernel
     has them too while dist_bucket has fewer than ATTN_MMA_X_MAX_DIST entries.  ``chunk`` > 0: a query sees
     only the keys of its own chunk of that many positions (chunks counted from position 0 of the
-    sequence); ``sink`` [nh] float32: exp(sink[h]) is added to the softmax denominator of head h."""
-    _attn_extras(nh, head_bias, dist_bias, dist_bucket, sink)
+    sequence); ``sink`` [nh] float32: exp(sink[h]) is added to the softmax denominator of head h;
+    ``slopes`` [nh] float32: slopes[h] * (i - j) is taken off the scaled score; ``temperature`` (coef, every):
+    the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)."""
+    _attn_extras(nh, head_bias, dist_bias, dist_bucket, sink, slopes)
     _check(lib().gg_attn_prefill_x(_p(q), ctypes.c_longlong(q_stride), _p(kcache), _p(vcache), dtype_code(kcache.dtype),
                                    _p(block_tables), bt_stride, _p(cu_q_lens), _p(context_lens), _p(tile_seq),
                                    _p(tile_q0), num_tiles, _p(tile64_seq), _p(tile64_q0), num_tiles64, int(allow_mma),
@@ -743,7 +763,7 @@ def attn_prefill_x(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcache:
                                    ctypes.c_float(softcap), int(keep_first), int(sigmoid_weights), _p(head_bias),
                                    _p(dist_bias), _p(dist_bucket),
                                    dist_bucket.numel() - 1 if dist_bucket is not None else 0, int(chunk or 0), _p(sink),
-                                   _stream()))
+                                   _p(slopes), *_temperature(temperature), _stream()))
 
 
 def attn_mma_x_chunk_sink() -> bool:
@@ -751,8 +771,15 @@ def attn_mma_x_chunk_sink() -> bool:
     return bool(lib().gg_attn_mma_x_chunk_sink())
 
 
-def _attn_extras(nh, head_bias, dist_bias, dist_bucket, sink=None) -> None:
-    _cuda(head_bias, dist_bias, dist_bucket, sink)
+def _temperature(temperature):
+    coef, every = temperature or (0.0, 0.0)
+    return ctypes.c_float(coef), ctypes.c_float(every)
+
+
+def _attn_extras(nh, head_bias, dist_bias, dist_bucket, sink=None, slopes=None) -> None:
+    _cuda(head_bias, dist_bias, dist_bucket, sink, slopes)
+    if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != nh):
+        raise KernelError("attention: the slopes are float32 [heads]")
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != nh):
         raise KernelError("attention: the sink is float32 [heads]")
     if head_bias is not None and (head_bias.dtype != torch.float32 or head_bias.numel() != nh):
@@ -769,9 +796,10 @@ def attn_decode_x(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcache: 
                   scale: float, softcap: float, allow_mma: bool = True, keep_first: int = 0,
                   sigmoid_weights: bool = False, head_bias: Optional[torch.Tensor] = None,
                   dist_bias: Optional[torch.Tensor] = None, dist_bucket: Optional[torch.Tensor] = None,
-                  chunk: int = 0, sink: Optional[torch.Tensor] = None) -> None:
+                  chunk: int = 0, sink: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
+                  temperature=None) -> None:
     """The same for single decoded tokens, split over the context and merged."""
-    _attn_extras(nh, head_bias, dist_bias, dist_bucket, sink)
+    _attn_extras(nh, head_bias, dist_bias, dist_bucket, sink, slopes)
     if part_o.numel() < n_dec * nh * num_splits * dv or part_ml.numel() < n_dec * nh * num_splits * 2:
         raise KernelError("attn_decode_x: scratch too small")
     _check(lib().gg_attn_decode_x(_p(q), ctypes.c_longlong(q_stride), _p(kcache), _p(vcache), dtype_code(kcache.dtype),
@@ -781,7 +809,7 @@ def attn_decode_x(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcache: 
                                   v_share, page_size, window, ctypes.c_float(scale), ctypes.c_float(softcap),
                                   int(allow_mma), int(keep_first), int(sigmoid_weights), _p(head_bias), _p(dist_bias),
                                   _p(dist_bucket), dist_bucket.numel() - 1 if dist_bucket is not None else 0,
-                                  int(chunk or 0), _p(sink), _stream()), 2)
+                                  int(chunk or 0), _p(sink), _p(slopes), *_temperature(temperature), _stream()), 2)
 
 
 def diff_combine(maps: torch.Tensor, out: torch.Tensor, lam: float, eps: float, post: float, heads: int,
@@ -892,12 +920,12 @@ def delta_recur(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, stat
                                 _stream()))
 
 
-def delta_out(o_raw: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, heads: int, dv: int,
+def delta_out(o_raw: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float, heads: int, dv: int,
               out: torch.Tensor, gate_act: str = "silu") -> None:
     """out[t, h] = o / sqrt(mean(o^2) + eps) * weight * act(gate[t, h]), act = silu or sigmoid; gate is
-    a column view [T, heads*dv] of a projection's output."""
+    a column view [T, heads*dv] of a projection's output; weight None: no weight."""
     _cuda(o_raw, weight, out)
-    if gate.stride(1) != 1 or gate.dtype != out.dtype or weight.dtype != torch.float32:
+    if gate.stride(1) != 1 or gate.dtype != out.dtype or weight is not None and weight.dtype != torch.float32:
         raise KernelError("delta_out: gate rows contiguous and of the output's dtype, float32 weight")
     _check(lib().gg_delta_out(_p(o_raw), _p(gate), ctypes.c_longlong(gate.stride(0)), dtype_code(out.dtype), _p(weight),
                               ctypes.c_float(eps), out.shape[0], heads, dv, {"silu": 0, "sigmoid": 1}[gate_act],
@@ -1119,3 +1147,18 @@ def mlstm_out(o_raw: torch.Tensor, m_row: torch.Tensor, gate: torch.Tensor, weig
     _check(lib().gg_mlstm_out(_p(o_raw), _p(m_row), _p(gate), ctypes.c_longlong(gate.stride(0)), dtype_code(out.dtype),
                               _p(weight), ctypes.c_float(eps), ctypes.c_float(floor), out.shape[0], heads, dv, dvp, _p(out),
                               _stream()))
+
+
+# ---------------------------------------------------------------- retention
+def retention_rows(x: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[torch.Tensor], interleaved: bool,
+                   heads: int, d: int, dv: int, kscale: float, out: torch.Tensor) -> None:
+    """Rows [q | k | v] of x (heads x d, heads x d, heads x dv) to float32 rows of the same layout: the first
+    2 * len(inv_freq) values of every q and k head rotated by the token's position, k times ``kscale``."""
+    _cuda(positions, inv_freq, out)
+    if x.stride(1) != 1 or out.dtype != torch.float32 or out.shape[1] != heads * (2 * d + dv) \
+            or (inv_freq is not None and inv_freq.dtype != torch.float64):
+        raise KernelError("retention_rows: contiguous rows in, float32 [T, heads * (2 d + dv)] out, float64 frequencies")
+    rot = 2 * inv_freq.numel() if inv_freq is not None else 0
+    _check(lib().gg_retention_rows(_p(x), ctypes.c_longlong(x.stride(0)), dtype_code(x.dtype), _p(positions), _p(inv_freq),
+                                   x.shape[0], heads, d, dv, rot, int(interleaved), ctypes.c_float(kscale), _p(out),
+                                   _stream()))

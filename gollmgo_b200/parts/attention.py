@@ -117,12 +117,16 @@ class Attention:
     """params: hidden_size, num_heads, num_kv_heads, head_dim, window (None = all
     keys), position (PartSpec); optional: v_head_dim (values of another size than keys),
     scale (of the scores; default head_dim^-1/2), softcap (scores pass cap * tanh(score / cap)),
+    distance_bias (bool: slope_h * (i - j) is taken off the scaled score, slope_h = 2^(-8 (h + 1) / heads)),
+    sink (bool: the softmax denominator has one more term exp(sink_h), a learned number a head, with no key and
+    no value; tensor ``sink_name``), temperature (coef, every): the query at position p is multiplied by
+    1 + coef * ln(floor((p + 1) / every) + 1),
     names (local names of the q, k, v, o tensors), out_buffer (name of the workspace buffer the
     result is left in, for a mixer that runs beside another).
 
-    Values of another size, shared value heads (``v_share``, set by a subclass) or capped
-    scores run on the general kernels (csrc/attention.cu: float32 arithmetic whatever the cache's
-    type); the tensor-core kernels take the plain case."""
+    Values of another size, shared value heads (``v_share``, set by a subclass), capped scores, a distance
+    bias, a sink or a temperature run on the general kernels (csrc/attention.cu: float32 arithmetic whatever the
+    cache's type) or their mma.sync form; the other tensor-core kernels take the plain case."""
 
     v_share = 1                  # consecutive key heads that read one value head
     bias = False                 # q, k, v and o have biases (local name + ".b")
@@ -143,10 +147,20 @@ class Attention:
         self.position = build_position(spec["position"], ctx)
         self.scale = float(spec.get("scale") or 1.0 / math.sqrt(self.d))
         self.softcap = float(spec.get("softcap") or 0.0)
+        self.has_sink = bool(spec.get("sink", False))
+        self.sink_name = spec.get("sink_name") or "sink"
+        self.temperature = tuple(float(v) for v in spec["temperature"]) if spec.get("temperature") else None
+        if self.temperature is not None and not self.temperature[1] > 0:
+            raise ValueError(f"a query temperature changes every {self.temperature[1]} positions")
+        self.slopes = self.sink = None
+        if spec.get("distance_bias"):
+            self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / self.nh) for h in range(self.nh)],
+                                       dtype=torch.float32, device=ctx.device)
         self.names = tuple(spec.get("names") or ("q_proj.weight", "k_proj.weight", "v_proj.weight", "o_proj.weight"))
         self.out_buffer = spec.get("out_buffer") or "mixer_out"
         self.nv = self.nkv // self.v_share
         self.general = (self.dv != self.d or self.softcap > 0 or self.v_share > 1 or self.bias or self.extras
+                        or self.has_sink or self.slopes is not None or self.temperature is not None
                         or float(getattr(self.position, "magnitude", 1.0)) != 1.0)
         self.qkv_width = (self.nh + self.nkv) * self.d + self.nv * self.dv
         self.qkv_bias = None
@@ -229,16 +243,21 @@ class Attention:
 
     def weights(self):
         q, k, v, o = self.names
-        return {q: WeightSpec((self.nh * self.d, self.hidden)),
-                k: WeightSpec((self.nkv * self.d, self.hidden)),
-                v: WeightSpec((self.nv * self.dv, self.hidden)),
-                o: WeightSpec((self.hidden, self.nh * self.dv))}
+        w = {q: WeightSpec((self.nh * self.d, self.hidden)),
+             k: WeightSpec((self.nkv * self.d, self.hidden)),
+             v: WeightSpec((self.nv * self.dv, self.hidden)),
+             o: WeightSpec((self.hidden, self.nh * self.dv))}
+        if self.has_sink:
+            w[self.sink_name] = WeightSpec((self.nh,), init="normal")
+        return w
 
     def load(self, get):
         q, k, v = (get(n) for n in self.names[:3])
         dt = torch.float32 if torch.float32 in (q.dtype, k.dtype, v.dtype) else q.dtype
         self.w_qkv = torch.cat([q.to(dt), k.to(dt), v.to(dt)], dim=0).contiguous()
         self.w_o = get(self.names[3]).contiguous()
+        if self.has_sink:
+            self.sink = get(self.sink_name).float().contiguous()
 
     # the optional protocol of parts/linear.py
     def takes_normed_rows(self, num_tokens):
@@ -291,6 +310,7 @@ class Attention:
                             self.d, self.nv, self.dv, self.ctx.page_size, self.position.interleaved, writes_cache)
         window = int(self.window or 0)
         bt = batch.block_tables[group]
+        more = dict(sink=self.sink, slopes=self.slopes, temperature=self.temperature)
         if batch.num_portions:
             if TILES_GENERAL not in batch.tiles:
                 raise RuntimeError("the step's batch was built without the index lists this mixer declares in "
@@ -300,7 +320,7 @@ class Attention:
                                t16.seq, t16.q0, t16.count, out, self.nh, self.nkv, self.d, self.dv, self.v_share,
                                self.ctx.page_size, window, self.scale, self.softcap,
                                t64.seq if t64 else None, t64.q0 if t64 else None, t64.count if t64 else 0,
-                               allow_mma=t64 is not None)
+                               allow_mma=t64 is not None, **more)
         if batch.num_decode:
             n = batch.num_decode
             facts = getattr(batch, "facts", None)
@@ -310,7 +330,7 @@ class Attention:
                               batch.dec_seqs, n, splits, ws.get("attn_part_o", 1, n * self.nh * splits * self.dv),
                               ws.get("attn_part_ml", 1, n * self.nh * splits * 2), out, self.nh, self.nkv, self.d,
                               self.dv, self.v_share, self.ctx.page_size, window, self.scale, self.softcap,
-                              allow_mma=self._mma_x)
+                              allow_mma=self._mma_x, **more)
         return out
 
     def forward(self, x, batch, cache, writes_cache=True, then=None):

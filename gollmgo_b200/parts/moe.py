@@ -15,12 +15,17 @@ experts and the weights the chosen scores divided by their sum (+ 1e-20); ``grou
 the experts form ``count`` equal groups of neighbours, a group's score is its best expert's, and
 only experts of the ``keep`` best groups can be chosen; ``activation="clamped_swish"`` (``limit``,
 ``alpha`` = 1.702, ``shift`` = 1): an expert computes g * sigmoid(alpha g) * (u + shift) with
-g = min(gate, limit), u = clamp(up, -limit, limit) instead of silu(gate) * up.
+g = min(gate, limit), u = clamp(up, -limit, limit) instead of silu(gate) * up;
+``router_weigh="sigmoid"``: the weights are the sigmoids of the chosen logits, not normalised;
+``weigh_input``: the weight multiplies the expert's input instead of its output (the first product is linear, so
+its results are multiplied in float32 before the activation and the input row is not rounded again);
+``shared_gate``: the shared expert's output is multiplied by sigmoid(w . x), one number a token (the row w is
+one more row of the router's product).
 
 params: hidden_size, intermediate_size, experts, top, router_bias (bool), router_weigh, groups,
-activation, limit, alpha, shift, shared (a feed-forward PartSpec or None), names: dict with "router",
-"router_bias", "expert" (a format string with {e}), "gate", "up", "down", "shared" (prefix of the
-shared expert's tensors).
+activation, limit, alpha, shift, weigh_input, shared (a feed-forward PartSpec or None), shared_gate, names: dict
+with "router", "router_bias", "expert" (a format string with {e}), "gate", "up", "down", "shared" (prefix of the
+shared expert's tensors), "shared_gate".
 """
 from __future__ import annotations
 
@@ -43,7 +48,7 @@ TC_TILE = 128
 ROUTE_LIB_TOKENS = int(os.environ.get("GOLLMGO_B200_MOE_ROUTE_LIB_TOKENS", "512"))
 
 DEFAULT_NAMES = {"router": "router", "router_bias": "router.b", "expert": "e{e}.", "gate": "gate",
-                 "up": "up", "down": "down", "shared": "shared."}
+                 "up": "up", "down": "down", "shared": "shared.", "shared_gate": "shared.sg"}
 
 
 class MixtureOfExperts:
@@ -74,15 +79,23 @@ class MixtureOfExperts:
             self.limit = float(spec["limit"])
             self.alpha = float(spec.get("alpha", 1.702))
             self.shift = float(spec.get("shift", 1.0))
+        self.weigh_input = bool(spec.get("weigh_input", False))
+        if self.weigh_input and self.activation != "silu":
+            raise ValueError("weights on the experts' input go with the silu-gated experts")
         self.names = {**DEFAULT_NAMES, **(spec.get("names") or {})}
         shared = spec.get("shared")
         self.shared = build_feed_forward(shared, ctx) if shared is not None else None
+        self.shared_gate = bool(spec.get("shared_gate", False)) and self.shared is not None
+        # the router's rows: one per expert, then the shared expert's gate, then (for a product whose rows
+        # start on 16-byte borders) rows of zeros
+        self.router_rows = -(-(self.experts + 1) // 8) * 8 if self.shared_gate else self.experts
         ws, T = ctx.workspace, ctx.max_tokens
         n = T * self.top
         self.tc_ok = (ctx.act_dtype == torch.bfloat16 and GEMM_POLICY != "lib" and self.hidden % 8 == 0
                       and self.inter % 8 == 0 and ctx.device.type == "cuda")
         slots = self._slots(n) if self.tc_ok and n >= TC_MIN_PAIRS else n
-        ws.reserve("moe_logits", T * self.experts, torch.float32)
+        ws.reserve("moe_logits", T * self.router_rows, torch.float32)
+        ws.reserve("moe_shared_gate", T, torch.float32)
         ws.reserve("moe_idx", n, torch.int32)
         ws.reserve("moe_wgt", n, torch.float32)
         ws.reserve("moe_order", slots, torch.int32)
@@ -114,10 +127,18 @@ class MixtureOfExperts:
             m[self._expert(e, "down")] = WeightSpec((self.hidden, self.inter))
         if self.shared is not None:
             m.update({self.names["shared"] + k: v for k, v in self.shared.weights().items()})
+        if self.shared_gate:
+            m[self.names["shared_gate"]] = WeightSpec((1, self.hidden))
         return m
 
     def load(self, get):
         self.w_router = get(self.names["router"]).contiguous()
+        if self.shared_gate:
+            w, sg = self.w_router, get(self.names["shared_gate"])
+            dt = torch.float32 if torch.float32 in (w.dtype, sg.dtype) else w.dtype
+            self.w_router = torch.zeros(self.router_rows, self.hidden, dtype=dt, device=w.device)
+            self.w_router[:self.experts] = w.to(dt)
+            self.w_router[self.experts:self.experts + 1] = sg.to(dt)
         self.b_router = get(self.names["router_bias"]).to(torch.float32).contiguous() if self.router_bias else None
         # [experts, 2 * inter, hidden]: an expert's gate rows, then its up rows
         self.w_gate_up = torch.stack([torch.cat([get(self._expert(e, "gate")), get(self._expert(e, "up"))], dim=0)
@@ -127,18 +148,24 @@ class MixtureOfExperts:
             self.shared.load(lambda local: get(self.names["shared"] + local))
 
     def route(self, x):
-        """(choices [T, top] int32, weights [T, top] float32) of the rows x."""
-        T, ws = x.shape[0], self.ctx.workspace
+        """(choices [T, top] int32, weights [T, top] float32, logits of the shared expert's gate [T, 1] or None)
+        of the rows x."""
+        T, ws, E = x.shape[0], self.ctx.workspace, self.experts
         idx, wgt = ws.get("moe_idx", T, self.top), ws.get("moe_wgt", T, self.top)
+        gate = None
         if T >= ROUTE_LIB_TOKENS and x.dtype == torch.bfloat16:
             # a long step: the logits are a product like any other (bfloat16 rows, float32 sums and result)
-            z = ws.get("moe_logits", T, self.experts)
+            z = ws.get("moe_logits", T, self.router_rows)
             linear(x, self.w_router, z)
-            ops.moe_topk(z, self.b_router, self.top, idx, wgt, self.weigh, self.group_count, self.group_keep)
+            ops.moe_topk(z, self.b_router, self.top, idx, wgt, self.weigh, self.group_count, self.group_keep, experts=E)
+            if self.shared_gate:
+                gate = z[:, E:E + 1]
         else:
-            ops.moe_route(x, self.w_router, self.b_router, self.top, idx, wgt, self.weigh, self.group_count,
-                          self.group_keep)
-        return idx, wgt
+            w = self.w_router
+            if self.shared_gate:
+                gate, w = ws.get("moe_shared_gate", T, 1), w[:E + 1]
+            ops.moe_route(x, w, self.b_router, self.top, idx, wgt, self.weigh, self.group_count, self.group_keep, gate=gate)
+        return idx, wgt, gate
 
     def _activate(self, gate_up, a):
         ops.clamped_gate(gate_up, a, self.limit, self.alpha, self.shift)
@@ -146,7 +173,8 @@ class MixtureOfExperts:
     def forward(self, x, batch):
         T, ws = x.shape[0], self.ctx.workspace
         n, E = T * self.top, self.experts
-        idx, wgt = self.route(x)
+        idx, wgt, sgate = self.route(x)
+        on_input = wgt if self.weigh_input else None
         place = ws.get("moe_place", 1, n)
         offsets = ws.get("moe_offsets", 1, E + 1)
         if self.tc_ok and n >= TC_MIN_PAIRS and x.is_contiguous():
@@ -158,7 +186,7 @@ class MixtureOfExperts:
             ops.moe_gather(x, order, self.top, xin)
             a = ws.get("moe_act", slots, self.inter)
             if self.activation == "silu":
-                ops.gemm_tc_grouped(xin, self.w_gate_up, a, tiles, E, gated=True)
+                ops.gemm_tc_grouped(xin, self.w_gate_up, a, tiles, E, gated=True, row_entry=order, row_scale=on_input)
             else:
                 gu = ws.get("moe_gate_up", slots, 2 * self.inter)
                 ops.gemm_tc_grouped(xin, self.w_gate_up, gu, tiles, E)
@@ -171,7 +199,7 @@ class MixtureOfExperts:
             a = ws.get("moe_act", n, self.inter)
             if self.activation == "silu":
                 ops.grouped_gemm(x, self.w_gate_up, a, self.inter, self.hidden, E, offsets=offsets, row_index=order,
-                                 row_div=self.top, rows=n, gated=True)
+                                 row_div=self.top, rows=n, gated=True, row_scale=on_input)
             else:
                 gu = ws.get("moe_gate_up", n, 2 * self.inter)
                 ops.grouped_gemm(x, self.w_gate_up, gu, 2 * self.inter, self.hidden, E, offsets=offsets, row_index=order,
@@ -181,7 +209,7 @@ class MixtureOfExperts:
             ops.grouped_gemm(a, self.w_down, y, self.hidden, self.inter, E, offsets=offsets, rows=n)
         shared = self.shared.forward(x, batch) if self.shared is not None else None
         out = ws.get("moe_out", T, self.hidden)
-        ops.moe_combine(y, place, wgt, shared, out, self.top)
+        ops.moe_combine(y, place, None if self.weigh_input else wgt, shared, out, self.top, gate=sgate)
         return out
 
 

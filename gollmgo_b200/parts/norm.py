@@ -16,20 +16,23 @@ from .registry import register_norm
 
 class RMSNorm:
     """params: size, eps, scalar (bool: the weight is one number for all coordinates; the kernels then
-    get it repeated ``size`` times)."""
+    get it repeated ``size`` times), offset (bool: the stored weight is what the factor differs from 1 by)."""
 
     def __init__(self, spec, ctx):
         self.size = int(spec["size"])
         self.eps = float(spec["eps"])
         self.scalar = bool(spec.get("scalar", False))
+        self.offset = bool(spec.get("offset", False))
         self.ctx = ctx
         self.weight = None
 
     def weights(self):
-        return {"": WeightSpec(() if self.scalar else (self.size,))}
+        return {"": WeightSpec(() if self.scalar else (self.size,), init="offset" if self.offset else "")}
 
     def load(self, get):
         w = get("").to(torch.float32)
+        if self.offset:
+            w = w + 1.0
         self.weight = (w.reshape(1).expand(self.size) if self.scalar else w).contiguous()
 
     def norm_in_place(self, resid):

@@ -3,7 +3,7 @@
 
 The value of a tensor depends only on (seed, tensor name, device kind), not on the
 order in which tensors are made.  Matrices and tables are N(0, std); norm weights
-are 1, or 1 + N(0, norm_jitter).
+are 1, or 1 + N(0, norm_jitter) (one less where the model stores them around zero).
 """
 from __future__ import annotations
 
@@ -37,7 +37,7 @@ def random_tensor(name: str, spec: WeightSpec, seed: int, device, dtype: torch.d
         t.uniform_(0.2, 0.8, generator=gen)
         return t.to(dtype)
     if len(spec.shape) <= 1 and spec.init != "normal":      # a norm's weight (a vector, or one number)
-        t = torch.ones(spec.shape, dtype=torch.float32, device=device)
+        t = (torch.zeros if spec.init == "offset" else torch.ones)(spec.shape, dtype=torch.float32, device=device)
         if norm_jitter:
             t += norm_jitter * torch.randn(spec.shape, generator=gen, dtype=torch.float32, device=device)
         return t.to(dtype)
