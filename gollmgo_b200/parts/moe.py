@@ -148,8 +148,11 @@ class MixtureOfExperts:
             self.shared.load(lambda local: get(self.names["shared"] + local))
 
     def route(self, x):
-        """(choices [T, top] int32, weights [T, top] float32, logits of the shared expert's gate [T, 1] or None)
-        of the rows x."""
+        """(choices [T, top] int32, weights [T, top] float32) of the rows x."""
+        return self._route(x)[:2]
+
+    def _route(self, x):
+        """route(x), and the logits of the shared expert's gate [T, 1] (None without one)."""
         T, ws, E = x.shape[0], self.ctx.workspace, self.experts
         idx, wgt = ws.get("moe_idx", T, self.top), ws.get("moe_wgt", T, self.top)
         gate = None
@@ -173,7 +176,7 @@ class MixtureOfExperts:
     def forward(self, x, batch):
         T, ws = x.shape[0], self.ctx.workspace
         n, E = T * self.top, self.experts
-        idx, wgt, sgate = self.route(x)
+        idx, wgt, sgate = self._route(x)
         on_input = wgt if self.weigh_input else None
         place = ws.get("moe_place", 1, n)
         offsets = ws.get("moe_offsets", 1, E + 1)

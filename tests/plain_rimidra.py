@@ -119,10 +119,14 @@ def choose(scores, top):
     return np.argsort(-scores, axis=-1, kind="stable")[:, :top]
 
 
-def mixture(h, w, p, f):
+def mixture(h, w, p, f, gaps=None):
+    """``gaps`` (a list): gets per token how far the last chosen score is above the best one left out."""
     T, top = h.shape[0], int(f["router"]["top"])
     s = sigmoid(h @ w[p + "router"].T)
     idx = choose(s, top)
+    if gaps is not None and top < s.shape[1]:
+        best = -np.sort(-s, axis=1)
+        gaps.append(best[:, top - 1] - best[:, top])
     out = np.zeros_like(h)
     for e in range(int(f["router"]["experts"])):
         t, j = np.nonzero(idx == e)
@@ -134,7 +138,7 @@ def mixture(h, w, p, f):
 
 
 # ---------------------------------------------------------------- the model
-def forward(cfg, w, tokens, return_layers=False):
+def forward(cfg, w, tokens, return_layers=False, gaps=None):
     """Logits [T, vocab] of one sequence; with ``return_layers`` also the stream after every layer."""
     eps = float(cfg["norm"]["eps"])
     x = w["embed"][np.asarray(tokens)]
@@ -150,7 +154,7 @@ def forward(cfg, w, tokens, return_layers=False):
         else:
             raise ValueError(layer["type"])
         if f is not None:
-            y = y + (dense(h, w, pre + "mlp.") if f["kind"] == "dense" else mixture(h, w, pre + "mlp.", f))
+            y = y + (dense(h, w, pre + "mlp.") if f["kind"] == "dense" else mixture(h, w, pre + "mlp.", f, gaps))
         x = x + y
         streams.append(x.copy())
     logits = offset_norm(x, w["final.norm"], eps) @ w["head"].T
