@@ -465,7 +465,8 @@ extern "C" int gg_attn_decode(const void* q, long long q_stride, const void* kca
 // gg_attn_decode with the work of gg_rope_kv_write for the same tokens folded in: q is the raw
 // projection output [T, (nh + 2 nkv) * d] (left as it is), the kernel rotates q and k with
 // half-split pairs over the whole head and writes k and v into the cache at slot_mapping[t]
-// (write_cache = 0: rotates q only).  bfloat16, head sizes 64 and 128, at most 16 heads per
+// (write_cache = 0: rotates q only).  Frequencies of zero turn nothing (a cosine of exactly 1): an attention
+// without rotation.  sink, slopes and the query temperature as in gg_attn_decode_x.  bfloat16, head sizes 64 and 128, at most 16 heads per
 // kv head; anything else is refused.
 extern "C" int gg_attn_decode_rope(const void* qkv, long long q_stride, void* kcache, void* vcache, int dtype,
                                    const int* block_tables, int bt_stride, const int* cu_q_lens,
@@ -473,6 +474,7 @@ extern "C" int gg_attn_decode_rope(const void* qkv, long long q_stride, void* kc
                                    float* part_o, float* part_ml, void* out, int nh, int nkv, int d,
                                    int page_size, int window, float scale, const int* positions,
                                    const int* slot_mapping, const double* inv_freq, int write_cache,
+                                   const float* sink, const float* slopes, float temp_coef, float temp_every,
                                    cudaStream_t stream) {
   AttnArgs a = {};
   a.q = qkv; a.q_stride = q_stride; a.kcache = kcache; a.vcache = vcache;
@@ -482,6 +484,7 @@ extern "C" int gg_attn_decode_rope(const void* qkv, long long q_stride, void* kc
   a.dec_seqs = dec_seqs; a.num_splits = num_splits; a.part_o = part_o; a.part_ml = part_ml;
   a.rope_inv_freq = inv_freq; a.rope_positions = positions; a.slot_mapping = slot_mapping;
   a.rope_write_cache = write_cache;
+  a.sink = sink; a.slopes = slopes; a.temp_coef = temp_coef; a.temp_every = temp_every;
   int rc = check_common(a, "attn_decode_rope");
   if (rc) return rc;
   GG_REQUIRE(n_dec >= 0 && num_splits >= 1 && num_splits <= 65535, "attn_decode_rope: bad n_dec %d or splits %d", n_dec, num_splits);

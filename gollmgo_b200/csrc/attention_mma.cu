@@ -338,7 +338,10 @@ __global__ void __launch_bounds__(MMA_THREADS, D == 128 ? 3 : 4) attn_decode_mma
                                       : (const __nv_bfloat16*)a.q + (size_t)t * a.q_stride + (size_t)head0 * D;
     load_q_frags<D>(qf, [&](int r) { return r < nrows ? qbase + (size_t)r * D : nullptr; });
     if (ROPE) __syncthreads();           // the loop's first copy lands where q was
-    const float sc = a.scale * LOG2E;
+    const float sc = a.scale * LOG2E * query_temperature(a, ctx - 1);
+    // rows g and g + 8 are heads head0 + g and head0 + g + 8 (clamped where the group is smaller)
+    const float slope0 = a.slopes ? a.slopes[head0 + min(g, nrows - 1)] * LOG2E : 0.f;
+    const float slope1 = a.slopes ? a.slopes[head0 + min(g + 8, nrows - 1)] * LOG2E : 0.f;
     for (int it = 0; it < ntiles; ++it) {
       const int nx = it + STAGES - 1;
       if (nx < ntiles) load_tile(nx, nx % STAGES);
@@ -359,6 +362,11 @@ __global__ void __launch_bounds__(MMA_THREADS, D == 128 ? 3 : 4) attn_decode_mma
           s[j][2] = tk < hi ? s[j][2] * sc : -INFINITY;
           s[j][1] = tk + 1 < hi ? s[j][1] * sc : -INFINITY;
           s[j][3] = tk + 1 < hi ? s[j][3] * sc : -INFINITY;
+          if (a.slopes) {
+            const float away = (float)(ctx - 1 - tk);
+            s[j][0] -= slope0 * away; s[j][2] -= slope1 * away;
+            s[j][1] -= slope0 * (away - 1.f); s[j][3] -= slope1 * (away - 1.f);
+          }
         }
         unsigned p[1][4];
         softmax_update<D, 2>(s, m, l, o, p);
@@ -451,6 +459,7 @@ __global__ void __launch_bounds__(MMA_THREADS, D == 128 ? 3 : 4) attn_decode_mma
             }
           }
         }
+        if (a.sink && M != -INFINITY) L += fast_exp2(fminf(a.sink[head0 + r] * LOG2E - M, 120.f));
         const float inv = L > 0.f ? 1.f / L : 0.f;
         *reinterpret_cast<unsigned*>(out + (size_t)r * D + col) = pack_bf16(o0 * inv, o1 * inv);
       }

@@ -204,10 +204,13 @@ def attn_decode_rope(qkv: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tens
                      part_o: torch.Tensor, part_ml: torch.Tensor, out: torch.Tensor, nh: int, nkv: int,
                      d: int, page_size: int, window: int, scale: float, positions: torch.Tensor,
                      slot_mapping: Optional[torch.Tensor], inv_freq: torch.Tensor,
-                     write_cache: bool = True) -> None:
+                     write_cache: bool = True, sink: Optional[torch.Tensor] = None,
+                     slopes: Optional[torch.Tensor] = None, temperature=None) -> None:
     """rope_kv_write and attn_decode of single decoded tokens in one kernel: qkv is the raw
-    projection output and stays as it is; k (rotated) and v land in the cache."""
+    projection output and stays as it is; k (rotated; frequencies of zero turn nothing) and v land in
+    the cache.  ``sink``, ``slopes`` and ``temperature`` as in attn_prefill_x."""
     _cuda(qkv, positions, slot_mapping, inv_freq, kcache, vcache)
+    _attn_extras(nh, None, None, None, sink, slopes)
     if not attn_decode_rope_ok(qkv.dtype, nh, nkv, d, inv_freq, False) or kcache.dtype != qkv.dtype:
         raise KernelError("attn_decode_rope: shape or dtype not taken (see attn_decode_rope_ok)")
     if qkv.shape[1] != (nh + 2 * nkv) * d or qkv.stride(0) != qkv.shape[1]:
@@ -221,7 +224,7 @@ def attn_decode_rope(qkv: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tens
                                      _p(cu_q_lens), _p(context_lens), _p(dec_seqs), n_dec, num_splits,
                                      _p(part_o), _p(part_ml), _p(out), nh, nkv, d, page_size, window,
                                      ctypes.c_float(scale), _p(positions), _p(slot_mapping), _p(inv_freq),
-                                     int(write_cache), _stream()), 2)
+                                     int(write_cache), _p(sink), _p(slopes), *_temperature(temperature), _stream()), 2)
 
 
 ATTN_FLAT_MAX_SEQS = 1024   # decoded tokens attn_decode_flat takes in one launch (FLAT_MAX_SEQS in attention_mma.cu)
@@ -1162,3 +1165,50 @@ def retention_rows(x: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[
     _check(lib().gg_retention_rows(_p(x), ctypes.c_longlong(x.stride(0)), dtype_code(x.dtype), _p(positions), _p(inv_freq),
                                    x.shape[0], heads, d, dv, rot, int(interleaved), ctypes.c_float(kscale), _p(out),
                                    _stream()))
+
+
+RETENTION_CHUNK = 64          # tokens of a chunk of the prompt kernels (RET_C in retention.cu)
+RETENTION_MAX_V = 512         # values of a head the chunk kernel takes
+
+
+def retention_scratch_floats(tokens: int, seqs: int, heads: int, d: int, dv: int) -> int:
+    return (tokens // RETENTION_CHUNK + seqs + 1) * heads * d * dv
+
+
+def retention_chunks(rows: torch.Tensor, log2_decay: torch.Tensor, state: torch.Tensor, scratch: torch.Tensor,
+                     tile_seq: torch.Tensor, tile_q0: torch.Tensor, num_tiles: int, cu_q_lens: torch.Tensor,
+                     context_lens: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, gate: torch.Tensor, eps: float,
+                     heads: int, d: int, dv: int, out: torch.Tensor) -> None:
+    """The tokens of prompt portions: S <- g S + k v^T, o = S^T q, out = o / sqrt(mean(o^2) + eps) * silu(gate), from
+    retention_rows' rows and from and to state [slots, heads, dv, d]; tiles of RETENTION_CHUNK rows (tile_seq, tile_q0)
+    are the chunks.  gate: a column view [T, heads*dv]; scratch float32 of retention_scratch_floats()."""
+    _cuda(rows, log2_decay, state, scratch, tile_seq, tile_q0, out)
+    T = rows.shape[0]
+    if rows.dtype != torch.float32 or rows.shape[1] != heads * (2 * d + dv) or log2_decay.dtype != torch.float32 \
+            or log2_decay.numel() != heads or state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dv, d) \
+            or scratch.dtype != torch.float32 or gate.stride(1) != 1 or gate.dtype != out.dtype:
+        raise KernelError("retention_chunks: float32 rows, decays, state [slots, heads, dv, d] and scratch; gate of the output's dtype")
+    _check(lib().gg_retention_states(_p(rows), _p(log2_decay), _p(state), _p(scratch), ctypes.c_longlong(scratch.numel()),
+                                     _p(cu_q_lens), _p(context_lens), _p(state_slots), T, num_seqs, heads, d, dv, _stream()))
+    _check(lib().gg_retention_chunks(_p(rows), _p(log2_decay), _p(scratch), _p(tile_seq), _p(tile_q0), num_tiles,
+                                     _p(cu_q_lens), _p(context_lens), _p(gate), ctypes.c_longlong(gate.stride(0)),
+                                     ctypes.c_float(eps), heads, d, dv, dtype_code(out.dtype), _p(out), _stream()))
+
+
+def retention_decode(proj: torch.Tensor, gate_col: int, positions: torch.Tensor, inv_freq: Optional[torch.Tensor],
+                     interleaved: bool, decay: torch.Tensor, state: torch.Tensor, dec_seqs: torch.Tensor, n_dec: int,
+                     cu_q_lens: torch.Tensor, context_lens: torch.Tensor, state_slots: torch.Tensor, heads: int, d: int,
+                     dv: int, kscale: float, eps: float, out: torch.Tensor) -> None:
+    """The same for single decoded tokens (the sequences dec_seqs), straight from the projection's rows
+    [q | k | v | .. | gate at gate_col]: rotation, step of the state, read-out, norm and gate in one kernel."""
+    _cuda(positions, inv_freq, decay, state, dec_seqs, out)
+    if proj.stride(1) != 1 or proj.dtype != out.dtype or decay.dtype != torch.float32 or decay.numel() != heads \
+            or state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dv, d) \
+            or (inv_freq is not None and inv_freq.dtype != torch.float64):
+        raise KernelError("retention_decode: rows of the output's dtype, float32 decays [heads] and state [slots, heads, dv, d], "
+                          "float64 frequencies")
+    rot = 2 * inv_freq.numel() if inv_freq is not None else 0
+    _check(lib().gg_retention_decode(_p(proj), ctypes.c_longlong(proj.stride(0)), int(gate_col), dtype_code(proj.dtype),
+                                     _p(positions), _p(inv_freq), _p(decay), _p(state), _p(dec_seqs), n_dec, _p(cu_q_lens),
+                                     _p(context_lens), _p(state_slots), heads, d, dv, rot, int(interleaved),
+                                     ctypes.c_float(kscale), ctypes.c_float(eps), _p(out), _stream()))

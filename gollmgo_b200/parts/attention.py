@@ -170,6 +170,14 @@ class Attention:
                        and ATTN_POLICY != "general" and self.qkv_width % 8 == 0)
         self.num_sms = torch.cuda.get_device_properties(ctx.device).multi_processor_count \
             if ctx.device.type == "cuda" else 148
+        # Steps of decoded tokens only: a bias by distance, a sink or a temperature on an attention that is plain
+        # otherwise run on the decode kernel that merges inside a cluster and writes the cache itself (which takes
+        # them as options; without a rotation it is given frequencies of zero).
+        plain = (self.dv == self.d and self.softcap == 0 and self.v_share == 1 and not self.bias and not self.extras
+                 and self.position.rope_table() is None and not hasattr(self.position, "apply"))
+        self._decode_fused = (self._mma_x and plain and FUSE_DECODE_ROPE and ctx.device.type == "cuda"
+                              and self.nh // self.nkv <= 16 and ctx.page_size & (ctx.page_size - 1) == 0)
+        self._no_turn = torch.zeros(self.d // 2, dtype=torch.float64, device=ctx.device) if self._decode_fused else None
         ws, T = ctx.workspace, ctx.max_tokens
         ws.reserve("qkv", T * self.qkv_width, ctx.act_dtype)
         ws.reserve("attn_out", T * self.nh * self.dv, ctx.act_dtype)
@@ -177,7 +185,7 @@ class Attention:
         gchunks = -(-(self.nh // self.nkv) // 16)
         self._ctas_per_split = self.nkv * gchunks
         self._cluster_cap = None
-        if ctx.device.type == "cuda" and not self.general:
+        if ctx.device.type == "cuda" and (not self.general or self._decode_fused):
             self._cluster_cap = [0] + [ops.attn_decode_cluster_capacity(ctx.act_dtype, self.d, s, self.nh // self.nkv)
                                        for s in range(1, ops.ATTN_MAX_CLUSTER + 1)]
         esize = torch.empty((), dtype=ctx.act_dtype).element_size()
@@ -305,6 +313,18 @@ class Attention:
         linear(x, self.w_qkv, qkv)
         if hasattr(self.position, "apply"):
             raise TypeError("a position encoding that rewrites q and k itself cannot be used with the general attention path")
+        if self._decode_fused and batch.num_decode and not batch.num_portions:
+            n = batch.num_decode
+            facts = getattr(batch, "facts", None)
+            longest = facts.max_context if facts is not None else max(s + q for s, q in zip(batch.q_starts, batch.q_lens))
+            splits = self._splits(n, longest)
+            ops.attn_decode_rope(qkv, kc, vc, batch.block_tables[group], batch.bt_stride, batch.cu_q_lens, batch.context_lens,
+                                 batch.dec_seqs, n, splits, ws.get("attn_part_o", 1, n * self.nh * splits * self.d),
+                                 ws.get("attn_part_ml", 1, n * self.nh * splits * 2), out, self.nh, self.nkv, self.d,
+                                 self.ctx.page_size, int(self.window or 0), self.scale, batch.positions,
+                                 batch.slot_mapping[group], self._no_turn, writes_cache, sink=self.sink, slopes=self.slopes,
+                                 temperature=self.temperature)
+            return out
         ops.rope_kv_write_x(qkv, batch.positions, batch.slot_mapping[group], self.position.rope_table(),
                             float(getattr(self.position, "magnitude", 1.0)), self.qkv_bias, kc, vc, self.nh, self.nkv,
                             self.d, self.nv, self.dv, self.ctx.page_size, self.position.interleaved, writes_cache)

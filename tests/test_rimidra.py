@@ -185,6 +185,24 @@ def test_attention_at_the_edges_of_the_window(kit, dtype, shape):
     close(got["b"], wb, dtype, **tol)
 
 
+@pytest.mark.parametrize("splits", [1, 2, 3, 8, 11])
+@pytest.mark.parametrize("shape", [(128, 4, 2, 64, 64, 200, (0.2, 40), 8), (136, 16, 1, 128, 128, 170, (0.1, 33), 16),
+                                   (96, 4, 2, 64, 128, 150, (0.2, 50), 16)])
+def test_decoded_tokens_over_slices_of_the_context(kit, shape, splits, monkeypatch):
+    """The context of a decoded token cut into any count of slices (merged inside a cluster up to eight, by a kernel
+    of its own beyond): the bias by distance and the temperature are every slice's, the sink enters once."""
+    import gollmgo_b200.parts.attention as attention
+    monkeypatch.setattr(attention, "FORCED_SPLITS", splits)
+    D, m, page = att_entry(shape)
+    w = att_weights(D, m, seed=45)
+    mixer = att_mixer(kit, torch.bfloat16, D, m, page)
+    mixer.load(lambda n: w[n].cuda().to(torch.bfloat16))
+    x = bf(torch.randn(300, D, generator=torch.Generator().manual_seed(46)))
+    want = torch.from_numpy(P.attention(x.numpy(), npw(w), "p.", m))
+    got = MixerRun(kit, mixer, torch.bfloat16, page).feed(x, [1] * 3 + cuts_of(257, [100]) + [1] * 40, "s")
+    close(got, want, torch.bfloat16, bf16=4e-2)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_the_first_tokens_of_a_sequence(kit, dtype):
     """Rows 0, 1, 2 have one, two, three keys: there the sink carries much of the weight, which a row of many keys
@@ -226,7 +244,8 @@ def ret_mixer(kit, dtype, D, m, eps, max_tokens=640):
 RET_SHAPES = [(64, 16, 24, (0.9, 0.97, 0.995), (8, 10000.0)), (128, 64, 64, (0.95, 0.999), (64, 1e6)), (100, 20, 11, (0.85, 1.0, 0.99), (6, 500.0)),
               (72, 9, 7, (0.93,), None), (192, 128, 160, (0.97, 0.998), (96, 10000.0)), (96, 32, 128, (0.6, 0.9, 0.99, 0.9995), (32, 10000.0)),
               (160, 200, 36, (0.99,), (40, 10000.0)), (128, 128, 256, (0.96875, 0.9921875), (128, 10000.0)), (64, 48, 96, (0.5, 0.8), (48, 100.0)),
-              (80, 256, 40, (0.98,), (256, 10000.0)), (64, 4, 300, (0.9, 0.99), (2, 50.0))]
+              (80, 256, 40, (0.98,), (256, 10000.0)), (64, 4, 300, (0.9, 0.99), (2, 50.0)),
+              (64, 8, 520, (0.9, 0.99), (8, 50.0))]
 
 
 def ret_entry(shape):
