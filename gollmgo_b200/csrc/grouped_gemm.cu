@@ -360,10 +360,226 @@ __global__ void __launch_bounds__(GGM_THREADS, 2) grouped_gemm_ring_kernel(Group
   }
 }
 
+// ---------------------------------------------------------------- few rows per group: streaming the weights
+// The experts' products of decoded tokens once more, as gemm_small_m.cu does a product of a few tokens: rows of W are
+// the M side of mma.sync m16n8k16 and a group's rows the N side (8 NT of them at a time), a lane copies 16-byte chunks
+// of its two rows of W into a private ring of shared memory several steps ahead and feeds each to the instruction, the
+// eight warps of a CTA take interleaved spans of K and are summed in a fixed order.  A CTA walks over units of GROUP
+// tiles of 16 rows of W (8 gate and 8 up rows if gated) of the groups that have rows, in steps of the grid, its ring
+// running across their borders; a group with more than 8 NT rows is walked once for every 8 NT of them.  Which groups
+// have rows is known on the device alone: every CTA makes the list from the offsets.
+#define GGS_WARPS 8
+#define GGS_THREADS (GGS_WARPS * 32)
+#define GGS_SPAN 64
+#define GGS_STAGES 5
+#define GGS_MAX_ENTRIES 256            // (group, first row) pairs with rows
+#define GGS_MAX_ROWS 1024
+
+template <bool GATED, int NT, int GROUP, int XB>
+__global__ void __launch_bounds__(GGS_THREADS, 2) grouped_stream_kernel(GroupedArgs a) {
+  constexpr int PASS = 8 * NT;
+  extern __shared__ __align__(16) unsigned char ggs_smem[];
+  uint4* ring = reinterpret_cast<uint4*>(ggs_smem);                                   // [warps][stages][4][32]
+  float (*red)[16][PASS + 1] = reinterpret_cast<float (*)[16][PASS + 1]>(ggs_smem + (size_t)GGS_WARPS * GGS_STAGES * 4 * 32 * 16);
+  int* arow_s = reinterpret_cast<int*>(red + GGS_WARPS);                              // [M]
+  float* scale_s = reinterpret_cast<float*>(arow_s + a.M);                            // [M]
+  __shared__ int ent_g[GGS_MAX_ENTRIES], ent_r[GGS_MAX_ENTRIES], ent_n[GGS_MAX_ENTRIES];
+  __shared__ int entries_s;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
+  const int N = a.N, K = a.K;
+  const int iters = K > warp * GGS_SPAN ? (K - warp * GGS_SPAN + GGS_WARPS * GGS_SPAN - 1) / (GGS_WARPS * GGS_SPAN) : 0;
+  const int tiles = GATED ? (N + 7) / 8 : (N + 15) / 16;                              // of one group
+  const int upe = (tiles + GROUP - 1) / GROUP;                                        // units of one list entry
+  const unsigned ring_base = smem_u32(ring) + (unsigned)((warp * GGS_STAGES * 4 * 32 + lane) * 16);
+  const __nv_bfloat16* A = (const __nv_bfloat16*)a.A;
+  const __nv_bfloat16* W = (const __nv_bfloat16*)a.W;
+  pdl_trigger();
+  pdl_wait();
+  if (warp == 0) {
+    int run = 0;
+    for (int e0 = 0; e0 < a.G; e0 += 32) {
+      const int e = e0 + lane;
+      const int lo = e < a.G ? a.offsets[e] : 0, hi = e < a.G ? a.offsets[e + 1] : 0;
+      const int cnt = (hi - lo + PASS - 1) / PASS;
+      int at = cnt;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) { const int v = __shfl_up_sync(0xffffffffu, at, o); if (lane >= o) at += v; }
+      const int total = __shfl_sync(0xffffffffu, at, 31);
+      at += run - cnt;
+      for (int i = 0; i < cnt; ++i)
+        if (at + i < GGS_MAX_ENTRIES) { ent_g[at + i] = e; ent_r[at + i] = lo + i * PASS; ent_n[at + i] = min(PASS, hi - lo - i * PASS); }
+      run += total;
+    }
+    if (lane == 0) entries_s = min(run, GGS_MAX_ENTRIES);
+  }
+  for (int r = threadIdx.x; r < a.M; r += GGS_THREADS) {
+    const int entry = a.row_index ? a.row_index[r] : r;
+    arow_s[r] = a.row_index ? entry / a.row_div : entry;
+    scale_s[r] = a.row_scale ? a.row_scale[entry] : 1.f;
+  }
+  __syncthreads();
+  const int units = entries_s * upe;
+  // CTAs start at different places of K and wrap around, so that they do not all ask for the same lines of A at once
+  const int rot = iters > 0 ? (int)(blockIdx.x % (unsigned)iters) : 0;
+  int p_unit = blockIdx.x, p_ki = 0, p_tj = 0, p_stage = 0, p_tile = 0, p_size = 0;
+  const __nv_bfloat16* p_w = W;
+  auto p_enter = [&]() {
+    if (p_unit < units) {
+      const int e = p_unit / upe;
+      p_tile = (p_unit - e * upe) * GROUP;
+      p_size = min(GROUP, tiles - p_tile);
+      p_w = W + (size_t)ent_g[e] * (GATED ? 2 : 1) * N * K;
+    }
+  };
+  p_enter();
+  auto issue = [&]() {
+    if (iters > 0 && p_unit < units) {
+      int n_a, n_b;
+      if (GATED) { n_a = (p_tile + p_tj) * 8 + g; n_b = n_a < N ? N + n_a : -1; if (n_a >= N) n_a = -1; }
+      else { n_a = (p_tile + p_tj) * 16 + g; n_b = n_a + 8; if (n_a >= N) n_a = -1; if (n_b >= N) n_b = -1; }
+      const int kk = p_ki + rot < iters ? p_ki + rot : p_ki + rot - iters;
+      const int k0 = (kk * GGS_WARPS + warp) * GGS_SPAN + c * 8, k1 = k0 + 32;
+      const unsigned dst = ring_base + (unsigned)(p_stage * 4 * 32 * 16);
+      const __nv_bfloat16* wa = p_w + (size_t)max(n_a, 0) * K;
+      const __nv_bfloat16* wb = p_w + (size_t)max(n_b, 0) * K;
+      cp_async16(dst, wa + min(k0, K - 8), (n_a >= 0 && k0 < K) ? 16 : 0);
+      cp_async16(dst + 512, wb + min(k0, K - 8), (n_b >= 0 && k0 < K) ? 16 : 0);
+      cp_async16(dst + 1024, wa + min(k1, K - 8), (n_a >= 0 && k1 < K) ? 16 : 0);
+      cp_async16(dst + 1536, wb + min(k1, K - 8), (n_b >= 0 && k1 < K) ? 16 : 0);
+      if (++p_tj == p_size) {
+        p_tj = 0;
+        if (++p_ki == iters) { p_ki = 0; p_unit += gridDim.x; p_enter(); }
+      }
+      p_stage = p_stage + 1 == GGS_STAGES ? 0 : p_stage + 1;
+    }
+    cp_async_commit();
+  };
+#pragma unroll
+  for (int s = 0; s < GGS_STAGES - 1; ++s) issue();
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  int c_stage = 0;
+  for (int unit = blockIdx.x; unit < units; unit += gridDim.x) {
+    const int e = unit / upe, tile0 = (unit - e * upe) * GROUP, gsize = min(GROUP, tiles - tile0);
+    const int r0 = ent_r[e], nrows = ent_n[e];
+    const __nv_bfloat16* xr[NT];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) xr[j] = g + 8 * j < nrows ? A + (size_t)arow_s[r0 + g + 8 * j] * a.lda : nullptr;
+    const int nt = (nrows + 7) >> 3;                   // how many of the NT column groups hold rows
+    float acc[GROUP][NT][4];
+#pragma unroll
+    for (int t = 0; t < GROUP; ++t)
+#pragma unroll
+      for (int j = 0; j < NT; ++j) { acc[t][j][0] = acc[t][j][1] = acc[t][j][2] = acc[t][j][3] = 0.f; }
+    for (int kb = 0; kb < iters; kb += XB) {
+      uint4 xb[XB][2 * NT];
+#pragma unroll
+      for (int u = 0; u < XB; ++u) {
+        const int ki = kb + u;
+        const int kk = ki + rot < iters ? ki + rot : ki + rot - iters;
+        const int k0 = (kk * GGS_WARPS + warp) * GGS_SPAN + c * 8, k1 = k0 + 32;
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          xb[u][2 * j] = (xr[j] && ki < iters && k0 < K) ? __ldg(reinterpret_cast<const uint4*>(xr[j] + k0)) : zero;
+          xb[u][2 * j + 1] = (xr[j] && ki < iters && k1 < K) ? __ldg(reinterpret_cast<const uint4*>(xr[j] + k1)) : zero;
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < XB; ++u) {
+        if (kb + u < iters) {
+#pragma unroll
+          for (int t = 0; t < GROUP; ++t) {
+            if (t < gsize) {
+              issue();
+              cp_async_wait<GGS_STAGES - 1>();
+              const uint4* st = ring + ((size_t)(warp * GGS_STAGES + c_stage) * 4) * 32 + lane;
+              const uint4 w0 = st[0], w1 = st[32], w2 = st[64], w3 = st[96];
+              c_stage = c_stage + 1 == GGS_STAGES ? 0 : c_stage + 1;
+#pragma unroll
+              for (int j = 0; j < NT; ++j) {
+                if (j < nt) {
+                  const uint4 x0 = xb[u][2 * j], x1 = xb[u][2 * j + 1];
+                  unsigned f[4];
+                  f[0] = w0.x; f[1] = w1.x; f[2] = w0.y; f[3] = w1.y;
+                  mma_bf16(acc[t][j], f, x0.x, x0.y);
+                  f[0] = w0.z; f[1] = w1.z; f[2] = w0.w; f[3] = w1.w;
+                  mma_bf16(acc[t][j], f, x0.z, x0.w);
+                  f[0] = w2.x; f[1] = w3.x; f[2] = w2.y; f[3] = w3.y;
+                  mma_bf16(acc[t][j], f, x1.x, x1.y);
+                  f[0] = w2.z; f[1] = w3.z; f[2] = w2.w; f[3] = w3.w;
+                  mma_bf16(acc[t][j], f, x1.z, x1.w);
+                }
+              }
+            }
+          }
+        }
+      }
+    }
+    // per tile: the warps' shares through shared memory, then the epilogue
+#pragma unroll
+    for (int t = 0; t < GROUP; ++t) {
+      if (t < gsize) {
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          if (j < nt) {
+            red[warp][g][8 * j + 2 * c] = acc[t][j][0];
+            red[warp][g][8 * j + 2 * c + 1] = acc[t][j][1];
+            red[warp][g + 8][8 * j + 2 * c] = acc[t][j][2];
+            red[warp][g + 8][8 * j + 2 * c + 1] = acc[t][j][3];
+          }
+        }
+        __syncthreads();
+        __nv_bfloat16* out = (__nv_bfloat16*)a.out;
+        if (GATED) {
+          for (int i = threadIdx.x; i < nrows * 8; i += GGS_THREADS) {
+            const int tok = i >> 3, r = i & 7, f = (tile0 + t) * 8 + r;
+            if (f < N) {
+              float gate = 0.f, up = 0.f;
+#pragma unroll
+              for (int w = 0; w < GGS_WARPS; ++w) { gate += red[w][r][tok]; up += red[w][r + 8][tok]; }
+              const float sc = scale_s[r0 + tok];
+              gate *= sc; up *= sc;
+              out[(size_t)(r0 + tok) * a.ldo + f] = __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+            }
+          }
+        } else {
+          for (int i = threadIdx.x; i < nrows * 16; i += GGS_THREADS) {
+            const int tok = i >> 4, r = i & 15, n = (tile0 + t) * 16 + r;
+            if (n < N) {
+              float v = 0.f;
+#pragma unroll
+              for (int w = 0; w < GGS_WARPS; ++w) v += red[w][r][tok];
+              out[(size_t)(r0 + tok) * a.ldo + n] = __float2bfloat16_rn(v * scale_s[r0 + tok]);
+            }
+          }
+        }
+        __syncthreads();
+      }
+    }
+  }
+  cp_async_wait<0>();
+}
+
+template <bool GATED, int NT, int GROUP, int XB>
+static int grouped_stream_go(const GroupedArgs& a, cudaStream_t stream) {
+  const size_t smem = (size_t)GGS_WARPS * GGS_STAGES * 4 * 32 * 16 + sizeof(float) * GGS_WARPS * 16 * (8 * NT + 1) + (size_t)a.M * 8;
+  static int num_sms = 0;
+  if (!num_sms) {
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess ||
+        cudaDeviceGetAttribute(&num_sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || num_sms <= 0)
+      num_sms = 148;
+  }
+  cudaError_t e = cudaFuncSetAttribute(grouped_stream_kernel<GATED, NT, GROUP, XB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return gg_fail(GG_ERR_CUDA, "grouped_gemm: %s", cudaGetErrorString(e));
+  gg_launch(grouped_stream_kernel<GATED, NT, GROUP, XB>, dim3(2 * num_sms), dim3(GGS_THREADS), smem, stream, a);
+  return gg_check_launch("grouped_gemm");
+}
+
+// max_rows: no group has more rows than this (0: not known).  It only chooses between kernels.
 extern "C" int gg_grouped_gemm(const void* A, long long lda, long long a_group_cols, const int* row_index,
                                int row_div, const void* W, void* out, long long ldo, long long o_group_cols,
                                const int* offsets, int M, int G, int N, int K, int Np, int gated,
-                               const void* gate, long long ldg, int gate_col0, const float* row_scale, int act_dtype,
+                               const void* gate, long long ldg, int gate_col0, const float* row_scale, int max_rows, int act_dtype,
                                cudaStream_t stream) {
   GG_REQUIRE(M >= 0 && G > 0 && N > 0 && K > 0 && Np >= N, "grouped_gemm: bad sizes M=%d G=%d N=%d K=%d Np=%d", M, G, N, K, Np);
   GG_REQUIRE(A && W && out, "grouped_gemm: a pointer is null");
@@ -386,6 +602,25 @@ extern "C" int gg_grouped_gemm(const void* A, long long lda, long long a_group_c
     else if (vec) gg_launch(grouped_gemm_kernel<T, false, BK, true>, grid, dim3(GGM_THREADS), 0, stream, a);           \
     else gg_launch(grouped_gemm_kernel<T, false, BK, false>, grid, dim3(GGM_THREADS), 0, stream, a);                   \
   } while (0)
+  static const bool stream_on = !(getenv("GOLLMGO_B200_GROUPED_STREAM") && getenv("GOLLMGO_B200_GROUPED_STREAM")[0] == '0');
+  if (act_dtype == GG_BF16 && vec && stream_on && offsets && !gate && a_group_cols == 0 && o_group_cols == 0 && Np == N &&
+      K >= 64 && M <= GGS_MAX_ROWS && M <= 20 * G && max_rows > 0) {
+    // rows a walk over a group's weights takes: enough for most groups of a step whose choices are spread by chance
+    // (8 experts of 4096 x 2048, gate and up: 24 tokens with two each 53 us in walks of 16 rows and 59 in walks of 24, 64
+    // tokens 77 and 66; beyond 20 rows a group on average the kernel with tiles of 32 rows is level)
+    const int pass = max_rows <= 8 ? 8 : M <= 10 * G ? 16 : 24;
+    if (G + M / pass <= GGS_MAX_ENTRIES) {
+      const bool many = (long long)G * (gated ? (N + 7) / 8 : (N + 15) / 16) >= 2048;     // enough tiles for units of two
+      if (gated) {
+        if (pass == 8) return many ? grouped_stream_go<true, 1, 2, 4>(a, stream) : grouped_stream_go<true, 1, 1, 4>(a, stream);
+        if (pass == 16) return many ? grouped_stream_go<true, 2, 2, 2>(a, stream) : grouped_stream_go<true, 2, 1, 4>(a, stream);
+        return many ? grouped_stream_go<true, 3, 2, 2>(a, stream) : grouped_stream_go<true, 3, 1, 2>(a, stream);
+      }
+      if (pass == 8) return many ? grouped_stream_go<false, 1, 2, 4>(a, stream) : grouped_stream_go<false, 1, 1, 4>(a, stream);
+      if (pass == 16) return many ? grouped_stream_go<false, 2, 2, 2>(a, stream) : grouped_stream_go<false, 2, 1, 4>(a, stream);
+      return many ? grouped_stream_go<false, 3, 2, 2>(a, stream) : grouped_stream_go<false, 3, 1, 2>(a, stream);
+    }
+  }
   static const bool ring_on = !(getenv("GOLLMGO_B200_GROUPED_RING") && getenv("GOLLMGO_B200_GROUPED_RING")[0] == '0');
   if (act_dtype == GG_BF16 && vec && K >= 4 * GGR_BK && ring_on) {
     const size_t smem = (size_t)GGR_STAGES * (GGM_BM + (gated ? 2 : 1) * GGM_BN) * GGR_LD * sizeof(__nv_bfloat16);

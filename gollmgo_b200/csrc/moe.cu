@@ -11,6 +11,10 @@
 //                 places of expert e in `sorted` (values t * top + j), `place` is the inverse
 // gg_moe_combine: out[t] = sum_j weight[t, j] * y[place[t * top + j]] (+ shared[t], times the sigmoid
 //                 of its gate where there is one), float32 sums in the order of j; no weights: plain sum
+// gg_parallel_join: what a block that runs a mixer and a feed-forward side by side does at its end, a CTA a token:
+//                 resid[t] += mult * (mixer[t] + bias + the sum gg_moe_combine makes), and, where the next norm is
+//                 given, h[t] = resid[t] / sqrt(mean(resid[t]^2) + eps) * w; with no experts (top = 0) `shared` is a
+//                 dense feed-forward's result
 // The products between them are gg_grouped_gemm's (grouped_gemm.cu).
 #include "common.cuh"
 
@@ -292,6 +296,70 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restri
   }
 }
 
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+}
+__device__ __forceinline__ void axpy4(float4& s, float w, float4 v) {
+  s.x = fmaf(w, v.x, s.x); s.y = fmaf(w, v.y, s.y); s.z = fmaf(w, v.z, s.z); s.w = fmaf(w, v.w, s.w);
+}
+
+template <typename TA>
+__global__ void parallel_join_kernel(float* __restrict__ resid, const TA* __restrict__ mixer, const TA* __restrict__ y,
+                                     const int* __restrict__ place, const float* __restrict__ wgt, int top,
+                                     const TA* __restrict__ shared_out, const float* __restrict__ gate, long long gate_stride,
+                                     const float* __restrict__ bias, float mult, const float* __restrict__ norm_w, float eps,
+                                     TA* __restrict__ h, int D, int vec) {
+  extern __shared__ __align__(16) float row[];       // [D]
+  __shared__ float red[33];
+  pdl_trigger();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const float sg = gate ? 1.f / (1.f + expf(-gate[t * gate_stride])) : 1.f;
+  float* x = resid + t * D;
+  float ss = 0.f;
+  if (vec) {
+    for (int c = threadIdx.x * 4; c < D; c += blockDim.x * 4) {
+      float4 s = load4(mixer + t * D + c), r = load4(x + c);
+      for (int j = 0; j < top; ++j)
+        axpy4(s, wgt ? wgt[t * top + j] : 1.f, load4(y + (size_t)place[t * top + j] * D + c));
+      if (shared_out) axpy4(s, sg, load4(shared_out + t * D + c));
+      if (bias) axpy4(s, 1.f, load4(bias + c));
+      axpy4(r, mult, s);
+      store4(x + c, r);
+      if (norm_w) { store4(row + c, r); ss += r.x * r.x + r.y * r.y + r.z * r.z + r.w * r.w; }
+    }
+  } else {
+    for (int c = threadIdx.x; c < D; c += blockDim.x) {
+      float s = to_f32(mixer[t * D + c]);
+      for (int j = 0; j < top; ++j)
+        s = fmaf(wgt ? wgt[t * top + j] : 1.f, to_f32(y[(size_t)place[t * top + j] * D + c]), s);
+      if (shared_out) s = fmaf(sg, to_f32(shared_out[t * D + c]), s);
+      if (bias) s += bias[c];
+      const float r = fmaf(mult, s, x[c]);
+      x[c] = r;
+      if (norm_w) { row[c] = r; ss += r * r; }
+    }
+  }
+  if (!norm_w) return;
+  const float f = rsqrtf(block_sum(ss, red) / (float)D + eps);
+  if (vec) {
+    for (int c = threadIdx.x * 4; c < D; c += blockDim.x * 4) {
+      const float4 r = load4(row + c), w = load4(norm_w + c);
+      store4(h + t * D + c, make_float4(r.x * f * w.x, r.y * f * w.y, r.z * f * w.z, r.w * f * w.w));
+    }
+  } else {
+    for (int c = threadIdx.x; c < D; c += blockDim.x) h[t * D + c] = from_f32<TA>(row[c] * f * norm_w[c]);
+  }
+}
+
 static int check_pick(const char* who, int E, int top, int weigh, int groups, int keep) {
   GG_REQUIRE(weigh >= 0 && weigh <= 2, "%s: unknown way %d of weighing the chosen experts", who, weigh);
   GG_REQUIRE(groups >= 1 && keep >= 1 && keep <= groups && E % groups == 0, "%s: %d experts in %d groups of which %d are kept", who, E, groups, keep);
@@ -312,7 +380,9 @@ extern "C" int gg_moe_route(const void* h, const void* wr, const float* bias, in
   const size_t smem = (size_t)tok * D * sizeof(float);
   GG_REQUIRE(smem <= 200 * 1024, "moe_route: rows of %d values do not fit in shared memory", D);
   const int vec = (act_dtype == GG_F32 ? D % 4 == 0 : D % 8 == 0) && ((size_t)wr % 16) == 0;
-  const int threads = E >= 8 ? 256 : 128;                  // at least ROUTE_TOK warps
+  // at least ROUTE_TOK warps; steps of a few tokens: a warp for every row of Wr where there are up to 32
+  const int wr_rows = E + (gate ? 1 : 0);
+  const int threads = tok == 1 && wr_rows > 8 ? (wr_rows < 32 ? wr_rows * 32 : 1024) : E >= 8 ? 256 : 128;
   const int blocks = (T + tok - 1) / tok;
 #define ROUTE_LAUNCH(T_, N_)                                                                                     \
   do {                                                                                                           \
@@ -383,4 +453,30 @@ extern "C" int gg_moe_combine(const void* y, const int* place, const float* wgt,
   else
     return gg_fail(GG_ERR_INVALID, "moe_combine: unknown dtype %d", act_dtype);
   return gg_check_launch("moe_combine");
+}
+
+extern "C" int gg_parallel_join(float* resid, const void* mixer, const void* y, const int* place, const float* wgt, int top,
+                                const void* shared_out, const float* gate, long long gate_stride, const float* bias, float mult,
+                                const float* norm_w, float eps, void* h, int T, int D, int act_dtype, cudaStream_t stream) {
+  GG_REQUIRE(T >= 0 && D > 0 && top >= 0, "parallel_join: bad sizes T=%d D=%d top=%d", T, D, top);
+  GG_REQUIRE(resid && mixer && (top == 0 || (y && place)) && (shared_out || !gate) && (h || !norm_w), "parallel_join: a pointer is null");
+  const size_t smem = norm_w ? (size_t)D * sizeof(float) : 0;
+  GG_REQUIRE(smem <= 200 * 1024, "parallel_join: rows of %d values do not fit in shared memory", D);
+  if (T == 0) return GG_OK;
+  const size_t at = (size_t)resid | (size_t)mixer | (size_t)y | (size_t)shared_out | (size_t)bias | (size_t)norm_w | (size_t)h;
+  const int vec = D % 4 == 0 && at % 16 == 0;
+  const int per = vec ? 4 : 1;
+  int threads = ((D + per - 1) / per + 31) / 32 * 32;
+  threads = threads > 512 ? 512 : threads;
+#define JOIN_LAUNCH(T_)                                                                                                          \
+  do {                                                                                                                           \
+    if (smem > 40 * 1024) cudaFuncSetAttribute(parallel_join_kernel<T_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    gg_launch(parallel_join_kernel<T_>, dim3(T), dim3(threads), smem, stream, resid, (const T_*)mixer, (const T_*)y, place, wgt, top, \
+              (const T_*)shared_out, gate, gate_stride, bias, mult, norm_w, eps, (T_*)h, D, vec);                                 \
+  } while (0)
+  if (act_dtype == GG_F32) JOIN_LAUNCH(float);
+  else if (act_dtype == GG_BF16) JOIN_LAUNCH(__nv_bfloat16);
+  else return gg_fail(GG_ERR_INVALID, "parallel_join: unknown dtype %d", act_dtype);
+#undef JOIN_LAUNCH
+  return gg_check_launch("parallel_join");
 }

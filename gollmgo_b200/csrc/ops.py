@@ -579,7 +579,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
                  a_group_cols: int = 0, o_group_cols: int = 0, n_padded: Optional[int] = None,
                  offsets: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None, row_div: int = 1,
                  rows: Optional[int] = None, gated: bool = False, gate: Optional[torch.Tensor] = None,
-                 gate_col0: int = 0, row_scale: Optional[torch.Tensor] = None) -> None:
+                 gate_col0: int = 0, row_scale: Optional[torch.Tensor] = None, max_rows: int = 0) -> None:
     """out_g = a_g @ w_g^T for every group g (csrc/grouped_gemm.cu).  w [groups, n (2n if gated), k].
     Without ``offsets`` every group has the first ``rows`` rows of a and reads columns
     g * a_group_cols .. + k of them; with ``offsets`` [groups + 1] group g has rows offsets[g] ..
@@ -587,7 +587,8 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
     of a.  Results go to out[r, g * o_group_cols : + n_padded] (zeros past n).  ``gate``: row r of
     group g is multiplied by sigmoid(gate[a row, gate_col0 + g]).  ``row_scale`` (float32): the products
     of row r are multiplied by row_scale[row_index[r]] (row_scale[r] without a row list) before the
-    activation: a factor on the input row that does not round it again."""
+    activation: a factor on the input row that does not round it again.  ``max_rows``: no group has more rows
+    than this (0: not known); few rows per group run on a kernel that streams the weights once."""
     _cuda(w, offsets, row_index, row_scale)
     if row_scale is not None and row_scale.dtype != torch.float32:
         raise KernelError("grouped_gemm: the factors on rows are float32")
@@ -600,7 +601,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
                                  int(row_div), _p(w), _p(out), ctypes.c_longlong(out.stride(0)),
                                  ctypes.c_longlong(o_group_cols), _p(offsets), M, groups, n, k,
                                  int(n_padded if n_padded is not None else n), int(gated), _p(gate),
-                                 ctypes.c_longlong(gate.stride(0) if gate is not None else 0), int(gate_col0), _p(row_scale),
+                                 ctypes.c_longlong(gate.stride(0) if gate is not None else 0), int(gate_col0), _p(row_scale), int(max_rows),
                                  dtype_code(a.dtype), _stream()))
 
 
@@ -702,6 +703,25 @@ def moe_combine(y: torch.Tensor, place: torch.Tensor, wgt: Optional[torch.Tensor
     T, D = out.shape
     _check(lib().gg_moe_combine(_p(y), _p(place), _p(wgt), _p(shared), _p(gate),
                                 ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _p(out), T, D, top, dtype_code(out.dtype), _stream()))
+
+
+def parallel_join(resid: torch.Tensor, mixer: torch.Tensor, mult: float, bias: Optional[torch.Tensor] = None,
+                  dense: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None,
+                  wgt: Optional[torch.Tensor] = None, top: int = 0, gate: Optional[torch.Tensor] = None,
+                  norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, normed: Optional[torch.Tensor] = None) -> None:
+    """resid[t] += mult * (mixer[t] + bias + sum_j wgt[t, j] * y[place[t * top + j]] + sigmoid(gate[t]) * dense[t]); every term
+    but the first is optional (wgt None: weights of 1, gate None: a factor of 1).  With ``norm_weight``: normed[t] =
+    resid[t] / sqrt(mean(resid[t]^2) + eps) * norm_weight."""
+    _cuda(resid, mixer, bias, dense, y, place, wgt, norm_weight, normed)
+    T, D = resid.shape
+    if resid.dtype != torch.float32 or mixer.shape != resid.shape \
+            or any(t is not None and (t.dtype != mixer.dtype or t.shape[-1] != D) for t in (dense, y, normed)) \
+            or any(t is not None and (t.dtype != torch.float32 or t.numel() != D) for t in (bias, norm_weight)) \
+            or (gate is not None and (gate.dtype != torch.float32 or gate.shape[0] != T)):
+        raise KernelError("parallel_join: float32 residual, rows of its width in the activation type, float32 bias, weight and gate")
+    _check(lib().gg_parallel_join(_p(resid), _p(mixer), _p(y), _p(place), _p(wgt), int(top), _p(dense), _p(gate),
+                                  ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _p(bias), ctypes.c_float(mult),
+                                  _p(norm_weight), ctypes.c_float(eps), _p(normed), T, D, dtype_code(mixer.dtype), _stream()))
 
 
 # ---------------------------------------------------------------- attention of any make (general kernels)

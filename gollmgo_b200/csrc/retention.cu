@@ -195,7 +195,7 @@ retention_states_kernel(const float* __restrict__ rows, const float* __restrict_
         vs[e] = (j < n && c0 + c < dv) ? vb[at + c] : 0.f;
       }
     }
-    if (tid < RET_C) wj[buf][tid] = exp2f(l2 * (float)(n - 1 - tid));      // (tokens past n hold zeros)
+    if (tid < RET_C) wj[buf][tid] = tid < n ? exp2f(l2 * (float)(n - 1 - tid)) : 0.f;
   };
   stage(0, 0);
   ret_commit();
@@ -227,18 +227,36 @@ retention_states_kernel(const float* __restrict__ rows, const float* __restrict_
     const float2 gn2 = make_float2(gn, gn);
 #pragma unroll
     for (int i = 0; i < 4; ++i) { S[i][0] = ret_mul2(S[i][0], gn2); S[i][1] = ret_mul2(S[i][1], gn2); }
-#pragma unroll 8
-    for (int j = 0; j < n; ++j) {
-      const float4 k4 = *reinterpret_cast<const float4*>(ks + j * RET_ST);
-      const float4 v4 = *reinterpret_cast<const float4*>(vs + j * RET_ST);
-      const float w = wj[buf][j];
-      const float2 va = ret_mul2(make_float2(v4.x, v4.y), make_float2(w, w)), vb2 = ret_mul2(make_float2(v4.z, v4.w), make_float2(w, w));
-      const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
+    // four tokens at a time, the next four read while these are worked on: there are few warps to hide the reads behind
+    float4 kn[4], vn[4];
+    float wn[4];
+    auto fetch = [&](int j0) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float2 k2 = make_float2(kk[i], kk[i]);
-        S[i][0] = ret_fma2(k2, va, S[i][0]);
-        S[i][1] = ret_fma2(k2, vb2, S[i][1]);
+      for (int u = 0; u < 4; ++u) {
+        kn[u] = *reinterpret_cast<const float4*>(ks + (j0 + u) * RET_ST);
+        vn[u] = *reinterpret_cast<const float4*>(vs + (j0 + u) * RET_ST);
+        wn[u] = wj[buf][j0 + u];
+      }
+    };
+    fetch(0);
+#pragma unroll 2
+    for (int j0 = 0; j0 < n; j0 += 4) {                // (tokens past n hold zeros)
+      float4 k4[4], v4[4];
+      float w[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) { k4[u] = kn[u]; v4[u] = vn[u]; w[u] = wn[u]; }
+      fetch(min(j0 + 4, RET_C - 4));
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float2 w2 = make_float2(w[u], w[u]);
+        const float2 va = ret_mul2(make_float2(v4[u].x, v4[u].y), w2), vc = ret_mul2(make_float2(v4[u].z, v4[u].w), w2);
+        const float kk[4] = {k4[u].x, k4[u].y, k4[u].z, k4[u].w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 k2 = make_float2(kk[i], kk[i]);
+          S[i][0] = ret_fma2(k2, va, S[i][0]);
+          S[i][1] = ret_fma2(k2, vc, S[i][1]);
+        }
       }
     }
     __syncthreads();                                 // the other buffer is refilled at the top of the next round
@@ -308,6 +326,7 @@ retention_chunks_kernel(const float* __restrict__ rows, const float* __restrict_
   stage(0, 0);
   ret_commit();
   if (vec) {
+#pragma unroll 4
     for (int e = tid; e < RET_C * (d >> 2); e += 256) {
       const int r = e & (RET_C - 1), c = (e >> 6) << 2;
       const float4 q4 = r < n ? *reinterpret_cast<const float4*>(rq + (size_t)r * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);

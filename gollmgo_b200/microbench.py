@@ -178,12 +178,16 @@ def sample(args) -> None:
 
 def grouped_gemm(args) -> None:
     """The products of a mixture of experts at decode size: --tokens tokens, each with --top of
-    --experts experts (choices spread evenly), width --hidden, experts' width --intermediate.  The
+    --experts experts (choices spread evenly, or with --random-choice drawn), width --hidden, experts' width --intermediate.  The
     bytes are the weights of the experts that got a row, read once; several copies of the weights
     are walked so that no launch finds them in L2."""
     T, E, top, D, F = args.tokens, args.experts, args.top, args.hidden, args.intermediate
     n = T * top
-    idx = (torch.arange(n, device="cuda", dtype=torch.int32) * 7 % E).contiguous()
+    if args.random_choice:
+        gen = torch.Generator().manual_seed(0)
+        idx = torch.rand(T, E, generator=gen).topk(top, dim=1).indices.to("cuda", torch.int32).reshape(-1).contiguous()
+    else:
+        idx = (torch.arange(n, device="cuda", dtype=torch.int32) * 7 % E).contiguous()
     used = len(set(idx.tolist()))
     offsets = torch.empty(E + 1, device="cuda", dtype=torch.int32)
     order, place = torch.empty(n, device="cuda", dtype=torch.int32), torch.empty(n, device="cuda", dtype=torch.int32)
@@ -196,8 +200,8 @@ def grouped_gemm(args) -> None:
     gu = [torch.randn(E, 2 * F, D, device="cuda", dtype=torch.bfloat16) * 0.02 for _ in range(copies)]
     dn = [torch.randn(E, D, F, device="cuda", dtype=torch.bfloat16) * 0.02 for _ in range(copies)]
     t1 = _time(lambda i: ops.grouped_gemm(x, gu[i % copies], a, F, D, E, offsets=offsets, row_index=order, row_div=top,
-                                          rows=n, gated=True), args.reps)
-    t2 = _time(lambda i: ops.grouped_gemm(a, dn[i % copies], y, D, F, E, offsets=offsets, rows=n), args.reps)
+                                          rows=n, gated=True, max_rows=T), args.reps)
+    t2 = _time(lambda i: ops.grouped_gemm(a, dn[i % copies], y, D, F, E, offsets=offsets, rows=n, max_rows=T), args.reps)
     b1, b2 = used * 2 * F * D * 2, used * D * F * 2
     print(f"grouped_gemm gate_up+silu  {n} pairs on {used} of {E} experts, {F}x{D}: {t1:7.1f} us  {b1 / t1 / 1e3:7.1f} GB/s")
     print(f"grouped_gemm down          {n} pairs on {used} of {E} experts, {D}x{F}: {t2:7.1f} us  {b2 / t2 / 1e3:7.1f} GB/s")
@@ -288,6 +292,7 @@ def main(argv=None) -> int:
     ap.add_argument("--experts", type=int, default=16, help="grouped_gemm: experts of the mixture")
     ap.add_argument("--top", type=int, default=2, help="grouped_gemm: experts a token")
     ap.add_argument("--shape", default="llama_3_1_8b", help="step_timeline: a file of bench_shapes/")
+    ap.add_argument("--random-choice", action="store_true", help="grouped_gemm: experts drawn at random instead of in turn")
     ap.add_argument("--prompt-tokens", type=int, default=0, help="step_timeline: a prompt step of so many tokens instead of a decode step")
     args = ap.parse_args(argv)
     if args.tokens is None:

@@ -89,6 +89,14 @@ class ResidualRows:
         self.rows = rows
 
 
+class PreparedNorm:
+    """What a block hands on when it has added everything to the residual stream and made the norm that the next
+    block starts with: ``rows`` is that norm's output."""
+
+    def __init__(self, rows):
+        self.rows = rows
+
+
 class PostNormBlock:
     """x += s1 * norm1(mixer(x)); x += s2 * norm2(ff(x)): the sublayers read the residual stream
     itself and the norms sit on what they return.  s1, s2 are per-channel scales ("layer scale":
@@ -151,8 +159,13 @@ class PostNormBlock:
 class ParallelBlock:
     """x += mult * (mixer(h) + ff(h)) with h = norm(x): one norm, and both sublayers read its
     output.  A layer without a feed-forward adds the mixer alone.  params: residual_mult (default 1).
-    The sum of the sublayers and the add to the stream are float32 (one kernel); a mixer that leaves
-    the bias of its output projection in ``deferred_bias`` has it added by the same kernel."""
+    The sum of the sublayers and the add to the stream are float32 (one kernel, csrc/moe.cu:
+    gg_parallel_join); a mixer that leaves the bias of its output projection in ``deferred_bias`` has it added by
+    the same kernel, a feed-forward that offers ``forward_pending`` (a mixture of experts) has its experts' results
+    summed there, and where the block that runs next is such a block too, the kernel also makes that block's norm
+    (the delta handed on is then its PreparedNorm)."""
+
+    chains_norms = True          # forward takes next_block=
 
     def __init__(self, layer_spec, mixer, feed_forward, mixer_norm, ffn_norm, ctx):
         self.mixer, self.feed_forward, self.mixer_norm, self.ctx = mixer, feed_forward, mixer_norm, ctx
@@ -162,18 +175,32 @@ class ParallelBlock:
         self.mult = float(layer_spec.block.get("residual_mult", 1.0))
         ctx.workspace.reserve("normed", ctx.max_tokens * self.hidden, ctx.act_dtype)
 
-    def forward(self, resid, delta, batch, cache, writes_cache=True):
+    def takes_normed_rows(self, T):
+        return False                                      # (the protocol of the pre-norm block; this one hands on PreparedNorm)
+
+    def forward(self, resid, delta, batch, cache, writes_cache=True, next_block=None):
         T = resid.shape[0]
-        if isinstance(delta, ResidualRows):
-            delta = None                                  # the block before has added everything itself
-        elif delta is not None and not torch.is_tensor(delta):
-            raise ValueError("a parallel block cannot take the norm's input from the block before it")
         h = self.ctx.workspace.get("normed", T, self.hidden)
-        self.mixer_norm.add_norm(resid, delta, h)
+        if isinstance(delta, PreparedNorm):
+            h = delta.rows
+        else:
+            if isinstance(delta, ResidualRows):
+                delta = None                              # the block before has added everything itself
+            elif delta is not None and not torch.is_tensor(delta):
+                raise ValueError("a parallel block cannot take the norm's input from the block before it")
+            self.mixer_norm.add_norm(resid, delta, h)
         a = self.mixer.forward(h, batch, cache, writes_cache)
-        f = self.feed_forward.forward(h, batch) if self.feed_forward is not None else None
-        ops.scaled_add(resid, a, f, self.mult, getattr(self.mixer, "deferred_bias", None))
-        return None
+        f = {}
+        if hasattr(self.feed_forward, "forward_pending"):
+            f = self.feed_forward.forward_pending(h, batch)
+        elif self.feed_forward is not None:
+            f = {"dense": self.feed_forward.forward(h, batch)}
+        nxt = getattr(next_block, "mixer_norm", None) if isinstance(next_block, ParallelBlock) else None
+        if nxt is not None and hasattr(nxt, "rms_weight_eps") and next_block.hidden == self.hidden:
+            w, eps = nxt.rms_weight_eps()
+            f.update(norm_weight=w, eps=eps, normed=h)    # over the rows both sublayers have read
+        ops.parallel_join(resid, a, self.mult, getattr(self.mixer, "deferred_bias", None), **f)
+        return PreparedNorm(h) if "normed" in f else None
 
 
 class SandwichBlock:

@@ -174,6 +174,14 @@ class MixtureOfExperts:
         ops.clamped_gate(gate_up, a, self.limit, self.alpha, self.shift)
 
     def forward(self, x, batch):
+        p = self.forward_pending(x, batch)
+        out = self.ctx.workspace.get("moe_out", x.shape[0], self.hidden)
+        ops.moe_combine(p["y"], p["place"], p["wgt"], p["dense"], out, p["top"], gate=p["gate"])
+        return out
+
+    def forward_pending(self, x, batch):
+        """The experts' results before they are summed per token, as the arguments of ``ops.parallel_join`` (a block
+        that adds them to the stream itself: parts/block.py)."""
         T, ws = x.shape[0], self.ctx.workspace
         n, E = T * self.top, self.experts
         idx, wgt, sgate = self._route(x)
@@ -202,18 +210,16 @@ class MixtureOfExperts:
             a = ws.get("moe_act", n, self.inter)
             if self.activation == "silu":
                 ops.grouped_gemm(x, self.w_gate_up, a, self.inter, self.hidden, E, offsets=offsets, row_index=order,
-                                 row_div=self.top, rows=n, gated=True, row_scale=on_input)
+                                 row_div=self.top, rows=n, gated=True, row_scale=on_input, max_rows=T)
             else:
                 gu = ws.get("moe_gate_up", n, 2 * self.inter)
                 ops.grouped_gemm(x, self.w_gate_up, gu, 2 * self.inter, self.hidden, E, offsets=offsets, row_index=order,
-                                 row_div=self.top, rows=n)
+                                 row_div=self.top, rows=n, max_rows=T)
                 self._activate(gu, a)
             y = ws.get("moe_rows", n, self.hidden)
-            ops.grouped_gemm(a, self.w_down, y, self.hidden, self.inter, E, offsets=offsets, rows=n)
+            ops.grouped_gemm(a, self.w_down, y, self.hidden, self.inter, E, offsets=offsets, rows=n, max_rows=T)
         shared = self.shared.forward(x, batch) if self.shared is not None else None
-        out = ws.get("moe_out", T, self.hidden)
-        ops.moe_combine(y, place, None if self.weigh_input else wgt, shared, out, self.top, gate=sgate)
-        return out
+        return {"y": y, "place": place, "wgt": None if self.weigh_input else wgt, "top": self.top, "dense": shared, "gate": sgate}
 
 
 register_feed_forward("moe", MixtureOfExperts)
