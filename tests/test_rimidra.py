@@ -384,6 +384,71 @@ def test_mixture_weighted_on_the_input(kit, dtype, experts, top, shared, T, D, F
         close(moe.forward(x[i:i + 1].cuda().to(dtype).contiguous(), None), want[i:i + 1], dtype)
 
 
+@pytest.mark.parametrize("rows", [[1, 0, 2, 0, 5, 0], [8, 9, 0, 16, 17, 1], [24, 25, 3, 0, 60, 0, 2, 7], [0, 0, 0, 0, 7, 0, 0, 0]])
+@pytest.mark.parametrize("N,K,groups_more", [(24, 64, 0), (41, 72, 0), (264, 1032, 0), (1000, 136, 24)])
+def test_products_that_stream_a_groups_weights(kit, rows, N, K, groups_more):
+    """Groups without rows, with one, with exactly a walk's rows and with more than one walk takes; features that are
+    no multiple of a tile; K shorter and longer than what the warps take in one round; units of one tile and of two
+    (many groups); factors on the rows before the activation; rows found through a list."""
+    g = torch.Generator().manual_seed(75)
+    rows = rows + [0] * groups_more
+    G, M, top = len(rows), sum(rows), 2
+    x = bf(torch.randn(M, K, generator=g))
+    w = bf(torch.randn(G, 2 * N, K, generator=g) / K ** 0.5)
+    order = torch.randperm(2 * M, generator=g)[:M].int()                     # row r reads x[order[r] // 2]
+    scale = torch.rand(2 * M, generator=g) + 0.3
+    offs = torch.tensor([0] + list(np.cumsum(rows)), dtype=torch.int32)
+    xs = x[order.long() // top] * scale.double()[order.long(), None]
+    gate, up, plain = torch.zeros(M, N).double(), torch.zeros(M, N).double(), torch.zeros(M, N).double()
+    for e in range(G):
+        lo, hi = int(offs[e]), int(offs[e + 1])
+        gate[lo:hi], up[lo:hi] = xs[lo:hi] @ w[e, :N].T, xs[lo:hi] @ w[e, N:].T
+        plain[lo:hi] = x[lo:hi] @ w[e, :N].T
+    xb, wb = x.cuda().bfloat16(), w.cuda().bfloat16()
+    most = max(rows)
+    out = torch.full((M, N), float("nan"), device="cuda", dtype=torch.bfloat16)
+    kit.ops.grouped_gemm(xb, wb, out, N, K, G, offsets=offs.cuda(), row_index=order.cuda(), row_div=top, rows=M, gated=True,
+                         row_scale=scale.float().cuda(), max_rows=most)
+    close(out, gate * torch.sigmoid(gate) * up, torch.bfloat16, bf16=1.2e-2)
+    one = wb[:, :N].contiguous()
+    for most in (most, 0):                                                   # 0: the kernel with tiles of 32 rows
+        out = torch.full((M, N), float("nan"), device="cuda", dtype=torch.bfloat16)
+        kit.ops.grouped_gemm(xb, one, out, N, K, G, offsets=offs.cuda(), rows=M, max_rows=most)
+        close(out, plain, torch.bfloat16, bf16=1.2e-2)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,D,top", [(1, 64, 1), (7, 100, 3), (33, 2048, 2), (5, 37, 0), (300, 256, 0)])
+def test_the_end_of_a_parallel_block(kit, dtype, T, D, top):
+    """Mixer, experts with and without weights, a gated dense result and a bias added to the stream with a factor, and
+    the next norm of the sum; every optional term left out in turn."""
+    g = torch.Generator().manual_seed(76)
+    r = lambda *s: bf(torch.randn(*s, generator=g))
+    resid, a, dense, y = torch.randn(T, D, generator=g), r(T, D), r(T, D), r(max(T * top, 1), D)
+    place = torch.randperm(T * top, generator=g).int() if top else None
+    wgt, gate = torch.rand(T, max(top, 1), generator=g), torch.randn(T, 8, generator=g)
+    bias, w = torch.randn(D, generator=g), torch.rand(D, generator=g) + 0.5
+    dev = lambda t: t.cuda().to(dtype).contiguous()
+    for use_w, use_gate, use_dense, use_bias, norm in ((1, 1, 1, 1, 1), (0, 1, 1, 0, 1), (1, 0, 1, 1, 0), (0, 0, 0, 0, 1)):
+        want = a.clone()
+        if top:
+            picked = y[place.long()].view(T, top, D)
+            want += (picked * (wgt.double()[:, :, None] if use_w else 1.0)).sum(1)
+        if use_dense:
+            want += dense * (torch.sigmoid(gate[:, 3:4].double()) if use_gate else 1.0)
+        if use_bias:
+            want += bias.double()
+        want = resid.double() + 0.7 * want
+        x, h = resid.clone().cuda(), torch.empty(T, D, device="cuda", dtype=dtype)
+        kit.ops.parallel_join(x, dev(a), 0.7, bias.cuda() if use_bias else None, dev(dense) if use_dense else None,
+                              dev(y) if top else None, place.cuda() if top else None, wgt.cuda() if top and use_w else None, top,
+                              gate.cuda()[:, 3:4] if use_gate and use_dense else None,
+                              **(dict(norm_weight=w.cuda(), eps=1e-3, normed=h) if norm else {}))
+        close(x, want, torch.float32, f32=2e-6)
+        if norm:
+            close(h, P.unit_rms(want.numpy(), 1e-3) * w.double().numpy(), dtype, f32=2e-6, bf16=8e-3)
+
+
 # ------------------------------------------------------------------ whole models through bin/trace_run
 LENGTHS = {"rim_a": [1, 5, 37, 70, 130, 96], "rim_b": [2, 64, 65, 231, 90, 33], "rim_c": [3, 66, 40, 150, 97, 29],
            "rim_d": [4, 17, 290, 33, 65, 140]}
