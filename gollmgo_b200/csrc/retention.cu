@@ -23,15 +23,59 @@ __device__ __forceinline__ void rotation_of(double pos, double inv_freq, float* 
   sincosf(r, s, c);
 }
 
-#define RET_HEADS 8          // heads (of q, k or v) a block of the rows kernel takes
+#define RET_HEADS 8          // heads (of q, k or v) a block of the element-wise rows kernel takes
 
-// grid (T, ceil(3H / 8)), 256 threads.  vec: four neighbouring values a thread (d, dv and the row stride multiples
-// of 4, rot a multiple of 8, half-split pairs, aligned rows)
+__device__ __forceinline__ float4 ret_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ret_load4(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
+// grid T, 256 threads: a token's whole row, four neighbouring values (of both halves of the rotated pairs) a thread.
+// d, dv and the row stride multiples of 4, rot a multiple of 8, half-split pairs, aligned rows.
+template <typename TA>
+__global__ void __launch_bounds__(256)
+retention_rows_vec_kernel(const TA* __restrict__ x, long long x_stride, const int* __restrict__ positions,
+                          const double* __restrict__ inv_freq, int H, int d, int dv, int rot, float kscale, float* __restrict__ out) {
+  extern __shared__ float cs[];                    // cos [rot/2], sin [rot/2]
+  pdl_trigger();
+  const size_t t = blockIdx.x;
+  const int half = rot >> 1;
+  for (int p = threadIdx.x; p < half; p += 256) rotation_of((double)positions[t], inv_freq[p], &cs[p], &cs[half + p]);
+  __syncthreads();
+  pdl_wait();
+  const TA* xr = x + t * x_stride;
+  float* o = out + t * (size_t)H * (2 * d + dv);
+  const int pairs = half >> 2, per = pairs + ((d - rot) >> 2);     // groups of a q or k head: turned pairs, then what passes
+  for (int e = threadIdx.x; e < 2 * H * per; e += 256) {
+    const int h = (unsigned)e / (unsigned)per, g = e - h * per;
+    const int base = h * d;
+    const float sc = h >= H ? kscale : 1.f;
+    if (g < pairs) {
+      const int c = g << 2;
+      const float4 a = ret_load4(xr + base + c), b = ret_load4(xr + base + half + c);
+      const float4 co = *reinterpret_cast<const float4*>(cs + c), si = *reinterpret_cast<const float4*>(cs + half + c);
+      *reinterpret_cast<float4*>(o + base + c) =
+          make_float4((a.x * co.x - b.x * si.x) * sc, (a.y * co.y - b.y * si.y) * sc, (a.z * co.z - b.z * si.z) * sc, (a.w * co.w - b.w * si.w) * sc);
+      *reinterpret_cast<float4*>(o + base + half + c) =
+          make_float4((b.x * co.x + a.x * si.x) * sc, (b.y * co.y + a.y * si.y) * sc, (b.z * co.z + a.z * si.z) * sc, (b.w * co.w + a.w * si.w) * sc);
+    } else {
+      const int c = rot + ((g - pairs) << 2);
+      const float4 a = ret_load4(xr + base + c);
+      *reinterpret_cast<float4*>(o + base + c) = make_float4(a.x * sc, a.y * sc, a.z * sc, a.w * sc);
+    }
+  }
+  const int v0 = 2 * H * d, nv = (H * dv) >> 2;
+  for (int e = threadIdx.x; e < nv; e += 256) *reinterpret_cast<float4*>(o + v0 + 4 * e) = ret_load4(xr + v0 + 4 * e);
+}
+
+// grid (T, ceil(3H / 8)), 256 threads, any sizes and either layout of the pairs
 template <typename TA>
 __global__ void __launch_bounds__(256)
 retention_rows_kernel(const TA* __restrict__ x, long long x_stride, const int* __restrict__ positions,
                       const double* __restrict__ inv_freq, int H, int d, int dv, int rot, int interleaved, float kscale,
-                      int vec, float* __restrict__ out) {
+                      float* __restrict__ out) {
   extern __shared__ float cs[];                    // cos [rot/2], sin [rot/2]
   pdl_trigger();
   const size_t t = blockIdx.x;
@@ -44,35 +88,6 @@ retention_rows_kernel(const TA* __restrict__ x, long long x_stride, const int* _
   const TA* xr = x + t * x_stride;
   float* o = out + t * C;
   const int wmax = max(d, dv);
-  if (vec) {
-    const int per = wmax >> 2;                     // groups of four values of a head (those past its size do nothing)
-    for (int e = threadIdx.x; e < (h1 - h0) * per; e += blockDim.x) {
-      const int h = h0 + e / per, c = (e % per) << 2;
-      const bool is_v = h >= 2 * H;
-      if (c >= (is_v ? dv : d)) continue;
-      const size_t base = is_v ? (size_t)2 * H * d + (size_t)(h - 2 * H) * dv : (size_t)h * d;
-      const float sc = h >= H && !is_v ? kscale : 1.f;
-      if (!is_v && c >= half && c < rot) continue; // the second half of the rotated pairs goes with the first
-      float a[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) a[j] = to_f32(xr[base + c + j]);
-      if (!is_v && c < half) {
-        float b[4], ra[4], rb[4];
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          b[j] = to_f32(xr[base + half + c + j]);
-          const float co = cs[c + j], si = cs[half + c + j];
-          ra[j] = (a[j] * co - b[j] * si) * sc;
-          rb[j] = (b[j] * co + a[j] * si) * sc;
-        }
-        *reinterpret_cast<float4*>(o + base + c) = make_float4(ra[0], ra[1], ra[2], ra[3]);
-        *reinterpret_cast<float4*>(o + base + half + c) = make_float4(rb[0], rb[1], rb[2], rb[3]);
-      } else {
-        *reinterpret_cast<float4*>(o + base + c) = make_float4(a[0] * sc, a[1] * sc, a[2] * sc, a[3] * sc);
-      }
-    }
-    return;
-  }
   for (int e = threadIdx.x; e < (h1 - h0) * wmax; e += blockDim.x) {
     const int h = h0 + e / wmax, c = e % wmax;
     const bool is_v = h >= 2 * H;
@@ -99,15 +114,20 @@ extern "C" int gg_retention_rows(const void* x, long long x_stride, int dtype, c
   GG_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= d && (rot == 0 || inv_freq), "retention_rows: %d rotated values of %d", rot, d);
   GG_REQUIRE((3 * H + RET_HEADS - 1) / RET_HEADS <= 65535 && rot <= 8192, "retention_rows: too many heads or rotated values");
   if (T == 0) return GG_OK;
-  const int vec = !interleaved && d % 4 == 0 && dv % 4 == 0 && rot % 8 == 0 && ((size_t)out % 16) == 0;
-  const dim3 grid(T, (3 * H + RET_HEADS - 1) / RET_HEADS);
+  GG_REQUIRE(dtype == GG_F32 || dtype == GG_BF16, "retention_rows: unknown dtype %d", dtype);
   const size_t smem = (size_t)rot * sizeof(float);
+  if (!interleaved && d % 4 == 0 && dv % 4 == 0 && rot % 8 == 0 && x_stride % 4 == 0 && ((size_t)out % 16) == 0 && ((size_t)x % 16) == 0) {
+    if (dtype == GG_F32)
+      gg_launch(retention_rows_vec_kernel<float>, dim3(T), dim3(256), smem, stream, (const float*)x, x_stride, positions, inv_freq, H, d, dv, rot, kscale, out);
+    else
+      gg_launch(retention_rows_vec_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, stream, (const __nv_bfloat16*)x, x_stride, positions, inv_freq, H, d, dv, rot, kscale, out);
+    return gg_check_launch("retention_rows");
+  }
+  const dim3 grid(T, (3 * H + RET_HEADS - 1) / RET_HEADS);
   if (dtype == GG_F32)
-    gg_launch(retention_rows_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, x_stride, positions, inv_freq, H, d, dv, rot, interleaved, kscale, vec, out);
-  else if (dtype == GG_BF16)
-    gg_launch(retention_rows_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, x_stride, positions, inv_freq, H, d, dv, rot, interleaved, kscale, vec, out);
+    gg_launch(retention_rows_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, x_stride, positions, inv_freq, H, d, dv, rot, interleaved, kscale, out);
   else
-    return gg_fail(GG_ERR_INVALID, "retention_rows: unknown dtype %d", dtype);
+    gg_launch(retention_rows_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, x_stride, positions, inv_freq, H, d, dv, rot, interleaved, kscale, out);
   return gg_check_launch("retention_rows");
 }
 
