@@ -32,6 +32,12 @@ __device__ __forceinline__ float4 ret_load4(const __nv_bfloat16* p) {
   return make_float4(lo.x, lo.y, hi.x, hi.y);
 }
 
+__device__ __forceinline__ void ret_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void ret_store4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+}
+
 // grid T, 256 threads: a token's whole row, four neighbouring values (of both halves of the rotated pairs) a thread.
 // d, dv and the row stride multiples of 4, rot a multiple of 8, half-split pairs, aligned rows.
 template <typename TA>
@@ -305,7 +311,7 @@ __global__ void __launch_bounds__(256, NV <= 2 ? 2 : 1)
 retention_chunks_kernel(const float* __restrict__ rows, const float* __restrict__ log2_decay, const float* __restrict__ scratch,
                         const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, const int* __restrict__ cu_q_lens,
                         const int* __restrict__ context_lens, const TA* __restrict__ gate, long long gate_stride, float eps,
-                        int H, int d, int dv, int vec, TA* __restrict__ out) {
+                        int H, int d, int dv, int vec, int vec_io, TA* __restrict__ out) {
   constexpr int VP = NV * 128;
   extern __shared__ __align__(16) float sm[];
   float* Qt = sm;                                    // [d][64]: q transposed
@@ -449,28 +455,45 @@ retention_chunks_kernel(const float* __restrict__ rows, const float* __restrict_
   ret_wait<0>();
   pdl_trigger();
   if (i0 >= n) return;
+  float ss[8];                                       // (columns past dv hold zeros)
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    float2 q = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int c = 0; c < 4 * NV; ++c) q = ret_fma2(acc[i][c], acc[i][c], q);
+    ss[2 * i] = q.x; ss[2 * i + 1] = q.y;
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
-    float o[4 * NV], ss = 0.f;
-#pragma unroll
-    for (int c = 0; c < 4 * NV; ++c) {
-      o[c] = (i & 1) ? acc[i >> 1][c].y : acc[i >> 1][c].x;        // (columns past dv hold zeros)
-      ss += o[c] * o[c];
-    }
-    const float f = rsqrtf(warp_sum(ss) / (float)dv + eps);
-    if (i0 + i >= n) continue;
+    if (i0 + i >= n) break;
+    const float f = rsqrtf(ss[i] / (float)dv + eps);
     const size_t t = (size_t)(t0 + q0 + i0 + i);
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
       const int col = j * 128 + lane * 4;
       const TA* gr = gate + t * gate_stride + (size_t)h * dv + col;
       TA* y = out + (t * H + h) * dv + col;
+      float o[4];
 #pragma unroll
-      for (int c = 0; c < 4; ++c)
-        if (col + c < dv) {
-          const float z = to_f32(gr[c]);
-          y[c] = from_f32<TA>(o[4 * j + c] * f * (z / (1.f + expf(-z))));
+      for (int c = 0; c < 4; ++c) o[c] = ((i & 1) ? acc[i >> 1][4 * j + c].y : acc[i >> 1][4 * j + c].x) * f;
+      if (vec_io) {
+        if (col < dv) {
+          const float4 z = ret_load4(gr);
+          ret_store4(y, make_float4(o[0] * (z.x / (1.f + expf(-z.x))), o[1] * (z.y / (1.f + expf(-z.y))),
+                                    o[2] * (z.z / (1.f + expf(-z.z))), o[3] * (z.w / (1.f + expf(-z.w)))));
         }
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+          if (col + c < dv) {
+            const float z = to_f32(gr[c]);
+            y[c] = from_f32<TA>(o[c] * (z / (1.f + expf(-z))));
+          }
+      }
     }
   }
 }
@@ -654,6 +677,7 @@ extern "C" int gg_retention_chunks(const float* rows, const float* log2_decay, c
   GG_REQUIRE(rows && log2_decay && scratch && gate && out && gate_stride >= (long long)H * dv, "retention_chunks: bad arguments");
   if (num_tiles == 0) return GG_OK;
   const int vec = d % 4 == 0 && dv % 4 == 0 && ((size_t)rows % 16) == 0 && ((size_t)scratch % 16) == 0;
+  const int vec_io = dv % 4 == 0 && gate_stride % 4 == 0 && ((size_t)gate % 16) == 0 && ((size_t)out % 16) == 0;
   const int NVv = dv <= 128 ? 1 : dv <= 256 ? 2 : 4;
   const int kt = d * RET_C > RET_C * RET_PT ? d * RET_C : RET_C * RET_PT;
   const size_t smem = (size_t)(d * RET_C + kt + 2 * RET_SLICE * NVv * 128) * sizeof(float);
@@ -662,7 +686,7 @@ extern "C" int gg_retention_chunks(const float* rows, const float* log2_decay, c
     cudaError_t e = cudaFuncSetAttribute(retention_chunks_kernel<TA, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     if (e != cudaSuccess) return gg_fail(GG_ERR_CUDA, "retention_chunks: %s", cudaGetErrorString(e));                         \
     gg_launch(retention_chunks_kernel<TA, NV>, dim3(num_tiles, H), dim3(256), smem, stream, rows, log2_decay, scratch, tile_seq, \
-              tile_q0, cu_q_lens, context_lens, (const TA*)gate, gate_stride, eps, H, d, dv, vec, (TA*)out);                  \
+              tile_q0, cu_q_lens, context_lens, (const TA*)gate, gate_stride, eps, H, d, dv, vec, vec_io, (TA*)out);                  \
   } while (0)
 #define RET_GO_NV(TA) do { if (NVv == 1) RET_GO(TA, 1); else if (NVv == 2) RET_GO(TA, 2); else RET_GO(TA, 4); } while (0)
   if (dtype == GG_F32) RET_GO_NV(float);
