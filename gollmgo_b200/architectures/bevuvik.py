@@ -12,7 +12,7 @@ from __future__ import annotations
 from ..config import register_architecture
 from ..config.bevuvik_config import BevuvikConfig, DiffAttentionConfig
 from ..parts.position import YarnScaling
-from ..parts.spec import LayerSpec, ModelSpec, PartSpec, RunEntry
+from ..parts.spec import LayerSpec, ModelSpec, PartSpec, looped_run_order
 
 
 def _position(rot, dim: int, interleaved: bool) -> PartSpec:
@@ -43,22 +43,10 @@ def _mixer(cfg: BevuvikConfig, m) -> PartSpec:
 
 
 def run_order(num_layers: int, loop) -> tuple:
-    """The layers in the order they run: those of the loop ``times`` times in a row, every pass
-    with cache entries of its own and the embedding output mixed in before its first layer."""
+    """The layers in the order they run, the loop's passes with the embedding output mixed in before each."""
     if loop is None:
-        return tuple(RunEntry(i, i) for i in range(num_layers))
-    order, cache = [], 0
-    for i in range(loop.start):
-        order.append(RunEntry(i, cache))
-        cache += 1
-    for _ in range(loop.times):
-        for i in range(loop.start, loop.stop):
-            order.append(RunEntry(i, cache, mix_input=(i == loop.start)))
-            cache += 1
-    for i in range(loop.stop, num_layers):
-        order.append(RunEntry(i, cache))
-        cache += 1
-    return tuple(order)
+        return looped_run_order(num_layers)
+    return looped_run_order(num_layers, loop.start, loop.stop, loop.times, mix_input=True)
 
 
 def bevuvik_spec(cfg: BevuvikConfig) -> ModelSpec:

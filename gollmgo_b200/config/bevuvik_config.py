@@ -86,6 +86,23 @@ class LoopConfig:
     times: int
 
 
+def read_loop(d: dict, num_layers: int) -> Optional[LoopConfig]:
+    """The run of layers that is repeated (``loop``: start, stop, times), or None."""
+    lp = d.get("loop")
+    if lp is None:
+        return None
+    if not isinstance(lp, dict):
+        raise ConfigError("config.json: 'loop' must be an object or null")
+    _only(lp, ("start", "stop", "times"), "loop")
+    start = lp.get("start")
+    if isinstance(start, bool) or not isinstance(start, int) or start < 0:
+        raise ConfigError(f"config.json: loop.start must be an integer >= 0, got {start!r}")
+    loop = LoopConfig(start, _int(lp, "stop", "loop"), _int(lp, "times", "loop"))
+    if not (loop.start < loop.stop <= num_layers):
+        raise ConfigError(f"config.json: loop {loop.start}..{loop.stop} does not lie inside the {num_layers} layers")
+    return loop
+
+
 @dataclass(frozen=True)
 class BevuvikConfig:
     vocab: int
@@ -129,25 +146,13 @@ class BevuvikConfig:
             else:
                 raise ConfigError(f"config.json: {where}.type {kind!r} is not known (known: attention, parallel)")
             layers.append(BevuvikLayerConfig(kind, mixer, _mlp(e.get("mlp"), where + ".mlp")))
-        loop = None
-        lp = d.get("loop")
-        if lp is not None:
-            if not isinstance(lp, dict):
-                raise ConfigError("config.json: 'loop' must be an object or null")
-            _only(lp, ("start", "stop", "times"), "loop")
-            start = lp.get("start")
-            if isinstance(start, bool) or not isinstance(start, int) or start < 0:
-                raise ConfigError(f"config.json: loop.start must be an integer >= 0, got {start!r}")
-            loop = LoopConfig(start, _int(lp, "stop", "loop"), _int(lp, "times", "loop"))
-            if not (loop.start < loop.stop <= len(layers)):
-                raise ConfigError(f"config.json: loop {loop.start}..{loop.stop} does not lie inside the {len(layers)} layers")
         eos = d.get("eos_token_id")
         eos_ids = () if eos is None else tuple(int(x) for x in (eos if isinstance(eos, (list, tuple)) else [eos]))
         mult = d.get("residual_mult", 1.0)
         if isinstance(mult, bool) or not isinstance(mult, (int, float)):
             raise ConfigError(f"config.json: residual_mult must be a number, got {mult!r}")
         return BevuvikConfig(vocab=_int(d, "vocab", "config"), width=_int(d, "width", "config"), eps=eps,
-                             residual_mult=float(mult), layers=tuple(layers), loop=loop,
+                             residual_mult=float(mult), layers=tuple(layers), loop=read_loop(d, len(layers)),
                              max_position_embeddings=int(d.get("max_position_embeddings", 1 << 17)),
                              eos_token_ids=eos_ids, bos_token_id=d.get("bos_token_id"))
 

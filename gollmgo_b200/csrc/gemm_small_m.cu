@@ -44,6 +44,7 @@ struct GsmFuse {
   // the gated product's activation: limit <= 0: silu(gate) * up; limit > 0: with g = min(gate, limit)
   // and u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + shift)
   float act_limit, act_alpha, act_shift;
+  int relu2;                  // GSM_OUT_BF16: the square of relu of the result
 };
 
 #define GSM_STAGES 6
@@ -264,6 +265,7 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ x, long long ldx,
 #pragma unroll
               for (int wv = 0; wv < GSM_WARPS; ++wv) v += red[wv][r][tok];
               if (fuse.in_partials) v *= row_scale[tok];
+              if (MODE == GSM_OUT_BF16 && fuse.relu2) { v = fmaxf(v, 0.f); v *= v; }
               if (MODE == GSM_OUT_F32) reinterpret_cast<float*>(out)[(size_t)tok * N + n] = v;
               else reinterpret_cast<__nv_bfloat16*>(out)[(size_t)tok * N + n] = __float2bfloat16_rn(v);
             }
@@ -283,7 +285,7 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ x, long long ldx,
 static int gemm_small_m_run(const void* x, long long ldx, const void* W, void* out, int M, int N,
                             int K, int mode, const float* in_partials, int in_tiles, int hidden,
                             float eps, float* resid, const float* norm_w, float* out_partials,
-                            float act_limit, float act_alpha, float act_shift, cudaStream_t stream) {
+                            float act_limit, float act_alpha, float act_shift, cudaStream_t stream, int relu2 = 0) {
   GG_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_small_m: bad sizes M=%d N=%d K=%d", M, N, K);
   GG_REQUIRE(M <= 16, "gemm_small_m: %d tokens; this kernel takes at most 16", M);
   GG_REQUIRE(K % 8 == 0 && ldx % 8 == 0, "gemm_small_m: K=%d and the row stride %lld of x must be multiples of 8", K, ldx);
@@ -296,7 +298,7 @@ static int gemm_small_m_run(const void* x, long long ldx, const void* W, void* o
   fuse.in_partials = in_partials; fuse.in_tiles = in_tiles;
   fuse.inv_h = hidden > 0 ? 1.0f / (float)hidden : 0.f; fuse.eps = eps;
   fuse.resid = resid; fuse.norm_w = norm_w; fuse.out_partials = out_partials;
-  fuse.act_limit = act_limit; fuse.act_alpha = act_alpha; fuse.act_shift = act_shift;
+  fuse.act_limit = act_limit; fuse.act_alpha = act_alpha; fuse.act_shift = act_shift; fuse.relu2 = relu2;
   const __nv_bfloat16* xp = (const __nv_bfloat16*)x;
   const __nv_bfloat16* wp = (const __nv_bfloat16*)W;
   const int num_tiles = mode == GSM_OUT_SILU ? (N + 7) / 8 : (N + 15) / 16;
@@ -352,6 +354,12 @@ extern "C" int gg_gemm_small_m_clamped(const void* x, long long ldx, const void*
                                        float limit, float alpha, float shift, cudaStream_t stream) {
   GG_REQUIRE(limit > 0.f, "gemm_small_m: the clamped activation needs a positive limit");
   return gemm_small_m_run(x, ldx, W, out, M, N, K, 2, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr, limit, alpha, shift, stream);
+}
+
+// out = the square of relu(x W^T), bfloat16.
+extern "C" int gg_gemm_small_m_relu2(const void* x, long long ldx, const void* W, void* out, int M, int N, int K,
+                                     cudaStream_t stream) {
+  return gemm_small_m_run(x, ldx, W, out, M, N, K, 0, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr, 0.f, 0.f, 0.f, stream, 1);
 }
 
 extern "C" int gg_gemm_small_m(const void* x, long long ldx, const void* W, void* out, int M, int N,

@@ -17,7 +17,7 @@
 //           store.
 // Epilogues: bfloat16; float32; SiLU-gated: columns [0,128) of the accumulator come
 // from the gate rows of W and [128,256) from the up rows of the same features, and
-// the tile written is silu(gate) * up (formula: kernels/gollmgo_ops.cu:361-374).
+// the tile written is silu(gate) * up (formula: kernels/gollmgo_ops.cu:361-374); the square of relu.
 // Rows of x beyond M, rows of W beyond N and columns beyond K are zero-filled by TMA;
 // the epilogue only stores what lies inside the output.
 //
@@ -30,7 +30,7 @@
 #define TC_BK 64
 #define TC_STAGES 4
 #define TC_THREADS 192
-enum { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_OUT_SILU = 2 };
+enum { TC_OUT_BF16 = 0, TC_OUT_F32 = 1, TC_OUT_SILU = 2, TC_OUT_RELU2 = 3 };
 enum { TC_ERR_EMPTY_WAIT = 1, TC_ERR_FULL_WAIT = 2, TC_ERR_ACC_WAIT = 3, TC_ERR_DRAIN = 4 };
 
 // A persistent CTA walks over output tiles blockIdx.x, blockIdx.x + gridDim.x, ...; tile t is
@@ -178,7 +178,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           tc_load32(tlane + c, r);
           float v[32];
 #pragma unroll
-          for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
+          for (int j = 0; j < 32; ++j) {
+            v[j] = __uint_as_float(r[j]);
+            if (MODE == TC_OUT_RELU2) { v[j] = fmaxf(v[j], 0.f); v[j] *= v[j]; }
+          }
           if (row < M) {
             if (MODE == TC_OUT_F32) store_row32(reinterpret_cast<float*>(out) + (size_t)row * N + n0 + c, v, N - (n0 + c));
             else store_row32(reinterpret_cast<__nv_bfloat16*>(out) + (size_t)row * N + n0 + c, v, N - (n0 + c));
@@ -230,7 +233,7 @@ int gg_make_map_2d(CUtensorMap* map, const void* ptr, int rows, int cols, long l
 }
 
 // mode: 0 = bfloat16 out [M, N]; 1 = float32 out [M, N]; 2 = W is [2N, K] (gate rows then up
-// rows), out is bfloat16 [M, N] = silu(x Wg^T) * (x Wu^T).  status: one int in device memory,
+// rows), out is bfloat16 [M, N] = silu(x Wg^T) * (x Wu^T); 3 = bfloat16 out, the square of relu(x W^T).  status: one int in device memory,
 // left untouched unless a wait inside the kernel ran out (then non-zero).
 static int gemm_tc_launch(const void* x, long long ldx, const void* W, void* out, int M, int N, int K,
                           int mode, int* status, int withhold_loads, cudaStream_t stream,
@@ -254,7 +257,7 @@ extern "C" int gg_gemm_tc_grouped(const void* x, long long ldx, const void* W, v
                                   const float* row_scale, int* status, cudaStream_t stream) {
   GG_REQUIRE(tile_group != nullptr && groups > 0, "gemm_tc_grouped: no groups given");
   GG_REQUIRE(M % TC_BM == 0, "gemm_tc_grouped: %d rows are no multiple of %d", M, TC_BM);
-  GG_REQUIRE(mode == TC_OUT_BF16 || mode == TC_OUT_SILU, "gemm_tc_grouped: mode %d", mode);
+  GG_REQUIRE(mode == TC_OUT_BF16 || mode == TC_OUT_SILU || mode == TC_OUT_RELU2, "gemm_tc_grouped: mode %d", mode);
   GG_REQUIRE(!row_scale || (row_entry && mode == TC_OUT_SILU), "gemm_tc_grouped: factors on rows go with the gated product and a row list");
   return gemm_tc_launch(x, ldx, W, out, M, N, K, mode, status, 0, stream, tile_group, groups, row_entry, row_scale);
 }
@@ -273,7 +276,7 @@ static int gemm_tc_launch(const void* x, long long ldx, const void* W, void* out
   GG_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_tc: bad sizes M=%d N=%d K=%d", M, N, K);
   GG_REQUIRE(K % 8 == 0 && ldx % 8 == 0, "gemm_tc: K=%d and the row stride %lld of x must be multiples of 8", K, ldx);
   GG_REQUIRE(((size_t)x % 16) == 0 && ((size_t)W % 16) == 0, "gemm_tc: x and W must be 16-byte aligned");
-  GG_REQUIRE(mode >= 0 && mode <= 2, "gemm_tc: unknown mode %d", mode);
+  GG_REQUIRE(mode >= 0 && mode <= 3, "gemm_tc: unknown mode %d", mode);
   GG_REQUIRE(mode != TC_OUT_SILU || N % 2 == 0, "gemm_tc: the gated product needs an even number of features");
   GG_REQUIRE(N % 2 == 0 || mode == TC_OUT_F32, "gemm_tc: bfloat16 rows of odd length are not 4-byte aligned");
   GG_REQUIRE(status != nullptr, "gemm_tc: no status word given");
@@ -312,6 +315,7 @@ static int gemm_tc_launch(const void* x, long long ldx, const void* W, void* out
   } while (0)
   if (mode == TC_OUT_BF16) TC_LAUNCH(TC_OUT_BF16);
   else if (mode == TC_OUT_F32) TC_LAUNCH(TC_OUT_F32);
+  else if (mode == TC_OUT_RELU2) TC_LAUNCH(TC_OUT_RELU2);
   else TC_LAUNCH(TC_OUT_SILU);
 #undef TC_LAUNCH
   if (e != cudaSuccess) return gg_fail(GG_ERR_CUDA, "gemm_tc: launch: %s", cudaGetErrorString(e));

@@ -8,7 +8,7 @@
 //                     [g * a_group_cols, g * a_group_cols + K) of it
 //   W_g:              [N, K] row-major ([2N, K] if gated: gate rows, then up rows) at W + g * rows * K
 //   out row r, columns [g * o_group_cols, g * o_group_cols + Np): the N results, then zeros
-//   epilogue:         gated: silu(x Wg^T) * (x Wu^T);   gate given: the row is multiplied by
+//   epilogue:         gated = 1: silu(x Wg^T) * (x Wu^T);   gated = 2: the square of relu(x W^T);   gate given: the row is multiplied by
 //                     sigmoid(gate[A row, gate_col0 + g])   (an output gate per head);
 //                     row_scale given: row r's products are multiplied by row_scale[row_index ? row_index[r] : r]
 //                     before the activation (a factor on the input row, without rounding the row again)
@@ -40,7 +40,7 @@ struct GroupedArgs {
   const void* W;
   void* out; long long ldo; long long o_group_cols;
   const int* offsets;
-  int M, G, N, K, Np, gated;
+  int M, G, N, K, Np, relu2;
   const void* gate; long long ldg; int gate_col0;
   const float* row_scale;
 };
@@ -213,6 +213,9 @@ __global__ void __launch_bounds__(GGM_THREADS, (sizeof(TA) == 2 ? (GATED ? 2 : 4
       if (GATED) {
         const float u = Cs1[r * GGM_LDC + c] * scale_s[r];
         v = v / (1.f + expf(-v)) * u;
+      } else if (a.relu2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
       }
       if (a.gate) {
         const float z = to_f32(((const TA*)a.gate)[(size_t)arow_s[r] * a.ldg + a.gate_col0 + g]);
@@ -350,6 +353,9 @@ __global__ void __launch_bounds__(GGM_THREADS, 2) grouped_gemm_ring_kernel(Group
       if (GATED) {
         const float u = Cs1[r * GGM_LDC + c] * scale_s[r];
         v = v / (1.f + expf(-v)) * u;
+      } else if (a.relu2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
       }
       if (a.gate) {
         const float z = to_f32(((const TA*)a.gate)[(size_t)arow_s[r] * a.ldg + a.gate_col0 + g]);
@@ -548,7 +554,9 @@ __global__ void __launch_bounds__(GGS_THREADS, 2) grouped_stream_kernel(GroupedA
               float v = 0.f;
 #pragma unroll
               for (int w = 0; w < GGS_WARPS; ++w) v += red[w][r][tok];
-              out[(size_t)(r0 + tok) * a.ldo + n] = __float2bfloat16_rn(v * scale_s[r0 + tok]);
+              v *= scale_s[r0 + tok];
+              if (a.relu2) { v = fmaxf(v, 0.f); v *= v; }
+              out[(size_t)(r0 + tok) * a.ldo + n] = __float2bfloat16_rn(v);
             }
           }
         }
@@ -578,17 +586,19 @@ static int grouped_stream_go(const GroupedArgs& a, cudaStream_t stream) {
 // max_rows: no group has more rows than this (0: not known).  It only chooses between kernels.
 extern "C" int gg_grouped_gemm(const void* A, long long lda, long long a_group_cols, const int* row_index,
                                int row_div, const void* W, void* out, long long ldo, long long o_group_cols,
-                               const int* offsets, int M, int G, int N, int K, int Np, int gated,
+                               const int* offsets, int M, int G, int N, int K, int Np, int act,
                                const void* gate, long long ldg, int gate_col0, const float* row_scale, int max_rows, int act_dtype,
                                cudaStream_t stream) {
   GG_REQUIRE(M >= 0 && G > 0 && N > 0 && K > 0 && Np >= N, "grouped_gemm: bad sizes M=%d G=%d N=%d K=%d Np=%d", M, G, N, K, Np);
   GG_REQUIRE(A && W && out, "grouped_gemm: a pointer is null");
   GG_REQUIRE(!row_index || row_div > 0, "grouped_gemm: a row list needs its divisor");
+  GG_REQUIRE(act >= 0 && act <= 2, "grouped_gemm: unknown activation %d", act);
   if (M == 0) return GG_OK;
+  const bool gated = act == 1;
   GroupedArgs a;
   a.A = A; a.lda = lda; a.a_group_cols = a_group_cols; a.row_index = row_index; a.row_div = row_div;
   a.W = W; a.out = out; a.ldo = ldo; a.o_group_cols = o_group_cols; a.offsets = offsets;
-  a.M = M; a.G = G; a.N = N; a.K = K; a.Np = Np; a.gated = gated;
+  a.M = M; a.G = G; a.N = N; a.K = K; a.Np = Np; a.relu2 = act == 2;
   a.gate = gate; a.ldg = ldg; a.gate_col0 = gate_col0; a.row_scale = row_scale;
   const int row_tiles = offsets ? (M + GGM_BM - 1) / GGM_BM + G : (M + GGM_BM - 1) / GGM_BM;
   GG_REQUIRE(row_tiles <= 65535 && G <= 65535, "grouped_gemm: %d row tiles or %d groups are too many for one launch", row_tiles, G);

@@ -6,11 +6,14 @@
 //                 the softmax over all experts renormalised over the chosen, or each chosen logit's
 //                 sigmoid as it is; optionally only experts of the best groups can be chosen (moe_pick);
 //                 optionally one more row of Wr, whose product with h[t] is left in gate[t] (the logit of a
-//                 shared expert's gate)
+//                 shared expert's gate); optionally the choice goes by softmax score + a correction per expert, and
+//                 the weights are multiplied by a factor
 // gg_moe_align:   the (token, choice) pairs sorted by expert: offsets[e] .. offsets[e+1] are the
-//                 places of expert e in `sorted` (values t * top + j), `place` is the inverse
+//                 places of expert e in `sorted` (values t * top + j), `place` is the inverse; choices
+//                 past the last expert (router outputs that stand for no tensors) get the place -1
 // gg_moe_combine: out[t] = sum_j weight[t, j] * y[place[t * top + j]] (+ shared[t], times the sigmoid
-//                 of its gate where there is one), float32 sums in the order of j; no weights: plain sum
+//                 of its gate where there is one), float32 sums in the order of j; no weights: plain sum; a
+//                 place of -1 reads same[t] (the experts' input) instead of a row of y
 // gg_parallel_join: what a block that runs a mixer and a feed-forward side by side does at its end, a CTA a token:
 //                 resid[t] += mult * (mixer[t] + bias + the sum gg_moe_combine makes), and, where the next norm is
 //                 given, h[t] = resid[t] / sqrt(mean(resid[t]^2) + eps) * w; with no experts (top = 0) `shared` is a
@@ -44,8 +47,10 @@ __device__ __forceinline__ void route_load(const __nv_bfloat16* w, float (&v)[8]
 // experts, weights = the chosen scores divided by their sum (+ 1e-20).  weigh = 2: weights = the sigmoid
 // of each chosen logit, not normalised (the largest sigmoids are the largest logits').  groups > 1: the experts form
 // that many equal groups of neighbours, a group's score is its best expert's, and only experts of the
-// `keep` best groups can be chosen.  Ties: the lower index.
-__device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, int groups, int keep, int lane,
+// `keep` best groups can be chosen.  corr (weigh = 1, one group): the choice goes by score + corr[e], the
+// weights are the scores alone.  The weights are multiplied by `scale`.  Ties: the lower index.
+__device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, int groups, int keep,
+                                         const float* __restrict__ corr, float scale, int lane,
                                          int* __restrict__ idx, float* __restrict__ wgt) {
   float zmax = 0.f, zsum = 1.f;
   if (weigh == 1) {
@@ -90,7 +95,8 @@ __device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, i
     float best = -INFINITY;
     int bi = 0x7fffffff;
     for (int e = lane; e < E; e += 32) {
-      const float v = zr[e];
+      float v = zr[e];
+      if (corr && v != -INFINITY) v = expf(v - zmax) / zsum + corr[e];     // -inf: chosen already
       if (v > best || (v == best && e < bi)) { best = v; bi = e; }
     }
 #pragma unroll
@@ -100,7 +106,8 @@ __device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, i
       if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
     }
     if (bi == 0x7fffffff) bi = 0;                    // every logit left is -inf or NaN
-    val[j] = best;
+    val[j] = corr ? zr[bi] : best;
+    __syncwarp();
     if (lane == 0) { idx[j] = bi; zr[bi] = -INFINITY; }
     __syncwarp();
   }
@@ -108,14 +115,14 @@ __device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, i
     if (weigh == 1) {
       float sum = 0.f;
       for (int j = 0; j < top; ++j) { val[j] = expf(val[j] - zmax) / zsum; sum += val[j]; }
-      for (int j = 0; j < top; ++j) wgt[j] = val[j] / (sum + 1e-20f);
+      for (int j = 0; j < top; ++j) wgt[j] = val[j] / (sum + 1e-20f) * scale;
     } else if (weigh == 2) {
-      for (int j = 0; j < top; ++j) wgt[j] = 1.f / (1.f + expf(-val[j]));
+      for (int j = 0; j < top; ++j) wgt[j] = scale / (1.f + expf(-val[j]));
     } else {
       const float m = val[0];                        // the largest comes first
       float sum = 0.f;
       for (int j = 0; j < top; ++j) { val[j] = expf(val[j] - m); sum += val[j]; }
-      for (int j = 0; j < top; ++j) wgt[j] = val[j] / sum;
+      for (int j = 0; j < top; ++j) wgt[j] = val[j] / sum * scale;
     }
   }
 }
@@ -123,6 +130,7 @@ __device__ __forceinline__ void moe_pick(float* zr, int E, int top, int weigh, i
 template <typename TA, int TOK>
 __global__ void moe_route_kernel(const TA* __restrict__ h, const TA* __restrict__ wr, const float* __restrict__ bias,
                                  int T, int D, int E, int top, int weigh, int groups, int keep,
+                                 const float* __restrict__ corr, float scale,
                                  int* __restrict__ idx, float* __restrict__ wgt, float* __restrict__ gate, int vec) {
   __shared__ float z[TOK][MOE_MAX_EXPERTS];
   extern __shared__ __align__(16) float xs[];              // TOK rows of D floats
@@ -174,13 +182,14 @@ __global__ void moe_route_kernel(const TA* __restrict__ h, const TA* __restrict_
   }
   __syncthreads();
   if (warp < nt)                                           // warp r picks for token t0 + r (the block has TOK warps or more)
-    moe_pick(z[warp], E, top, weigh, groups, keep, lane, idx + (size_t)(t0 + warp) * top, wgt + (size_t)(t0 + warp) * top);
+    moe_pick(z[warp], E, top, weigh, groups, keep, corr, scale, lane, idx + (size_t)(t0 + warp) * top, wgt + (size_t)(t0 + warp) * top);
 }
 
 // The choice alone, from logits a product has already made (long steps: z = h Wr^T in float32 by the
 // vendor library from the bfloat16 rows): one warp a token adds the bias, picks and weighs.
 __global__ void moe_topk_kernel(const float* __restrict__ z, long long z_stride, const float* __restrict__ bias, int T, int E, int top,
-                                int weigh, int groups, int keep, int* __restrict__ idx, float* __restrict__ wgt) {
+                                int weigh, int groups, int keep, const float* __restrict__ corr, float scale,
+                                int* __restrict__ idx, float* __restrict__ wgt) {
   extern __shared__ float zs[];                            // warps x E
   pdl_trigger();
   pdl_wait();
@@ -190,7 +199,7 @@ __global__ void moe_topk_kernel(const float* __restrict__ z, long long z_stride,
   float* zr = zs + warp * E;
   for (int e = lane; e < E; e += 32) zr[e] = z[t * z_stride + e] + (bias ? bias[e] : 0.f);
   __syncwarp();
-  moe_pick(zr, E, top, weigh, groups, keep, lane, idx + (size_t)t * top, wgt + (size_t)t * top);
+  moe_pick(zr, E, top, weigh, groups, keep, corr, scale, lane, idx + (size_t)t * top, wgt + (size_t)t * top);
 }
 
 // One CTA.  counts and cursors in shared memory; the order of the rows inside an expert's range
@@ -209,7 +218,8 @@ __global__ void moe_align_kernel(const int* __restrict__ idx, int n, int E, int 
   if (pad > 1)
     for (int i = threadIdx.x; i < slots; i += blockDim.x) sorted[i] = -1;
   __syncthreads();
-  for (int i = threadIdx.x; i < n; i += blockDim.x) atomicAdd(&cnt[idx[i]], 1);
+  for (int i = threadIdx.x; i < n; i += blockDim.x)
+    if (idx[i] < E) atomicAdd(&cnt[idx[i]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int run = 0;
@@ -233,6 +243,7 @@ __global__ void moe_align_kernel(const int* __restrict__ idx, int n, int E, int 
       tile_group[i] = g;
     }
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    if (idx[i] >= E) { place[i] = -1; continue; }
     const int p = atomicAdd(&cnt[idx[i]], 1);
     sorted[p] = i;
     place[i] = p;
@@ -260,10 +271,17 @@ __global__ void moe_gather_kernel(const TA* __restrict__ x, const int* __restric
   }
 }
 
+// The row that choice i of token t adds.
+template <typename TA>
+__device__ __forceinline__ const TA* moe_row(const TA* y, const int* place, const TA* same, size_t t, size_t i, int D) {
+  const int p = place[i];
+  return p >= 0 ? y + (size_t)p * D : same + t * D;
+}
+
 template <typename TA>
 __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restrict__ place, const float* __restrict__ wgt,
                                    const TA* __restrict__ shared_out, const float* __restrict__ gate, long long gate_stride,
-                                   TA* __restrict__ out, int D, int top) {
+                                   const TA* __restrict__ same, TA* __restrict__ out, int D, int top) {
   pdl_trigger();
   pdl_wait();
   const size_t t = blockIdx.x;
@@ -273,7 +291,7 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restri
       float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
       for (int j = 0; j < top; ++j) {
         const float w = wgt ? wgt[t * top + j] : 1.f;
-        const TA* r = y + (size_t)place[t * top + j] * D + c;
+        const TA* r = moe_row(y, place, same, t, t * top + j, D) + c;
         s0 = fmaf(w, to_f32(r[0]), s0); s1 = fmaf(w, to_f32(r[1]), s1);
         s2 = fmaf(w, to_f32(r[2]), s2); s3 = fmaf(w, to_f32(r[3]), s3);
       }
@@ -290,7 +308,7 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restri
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     float s = 0.f;
     for (int j = 0; j < top; ++j)
-      s = fmaf(wgt ? wgt[t * top + j] : 1.f, to_f32(y[(size_t)place[t * top + j] * D + c]), s);
+      s = fmaf(wgt ? wgt[t * top + j] : 1.f, to_f32(moe_row(y, place, same, t, t * top + j, D)[c]), s);
     if (shared_out) s = fmaf(sg, to_f32(shared_out[t * D + c]), s);
     out[t * D + c] = from_f32<TA>(s);
   }
@@ -315,7 +333,7 @@ template <typename TA>
 __global__ void parallel_join_kernel(float* __restrict__ resid, const TA* __restrict__ mixer, const TA* __restrict__ y,
                                      const int* __restrict__ place, const float* __restrict__ wgt, int top,
                                      const TA* __restrict__ shared_out, const float* __restrict__ gate, long long gate_stride,
-                                     const float* __restrict__ bias, float mult, const float* __restrict__ norm_w, float eps,
+                                     const TA* __restrict__ same, const float* __restrict__ bias, float mult, const float* __restrict__ norm_w, float eps,
                                      TA* __restrict__ h, int D, int vec) {
   extern __shared__ __align__(16) float row[];       // [D]
   __shared__ float red[33];
@@ -329,7 +347,7 @@ __global__ void parallel_join_kernel(float* __restrict__ resid, const TA* __rest
     for (int c = threadIdx.x * 4; c < D; c += blockDim.x * 4) {
       float4 s = load4(mixer + t * D + c), r = load4(x + c);
       for (int j = 0; j < top; ++j)
-        axpy4(s, wgt ? wgt[t * top + j] : 1.f, load4(y + (size_t)place[t * top + j] * D + c));
+        axpy4(s, wgt ? wgt[t * top + j] : 1.f, load4(moe_row(y, place, same, t, t * top + j, D) + c));
       if (shared_out) axpy4(s, sg, load4(shared_out + t * D + c));
       if (bias) axpy4(s, 1.f, load4(bias + c));
       axpy4(r, mult, s);
@@ -340,7 +358,7 @@ __global__ void parallel_join_kernel(float* __restrict__ resid, const TA* __rest
     for (int c = threadIdx.x; c < D; c += blockDim.x) {
       float s = to_f32(mixer[t * D + c]);
       for (int j = 0; j < top; ++j)
-        s = fmaf(wgt ? wgt[t * top + j] : 1.f, to_f32(y[(size_t)place[t * top + j] * D + c]), s);
+        s = fmaf(wgt ? wgt[t * top + j] : 1.f, to_f32(moe_row(y, place, same, t, t * top + j, D)[c]), s);
       if (shared_out) s = fmaf(sg, to_f32(shared_out[t * D + c]), s);
       if (bias) s += bias[c];
       const float r = fmaf(mult, s, x[c]);
@@ -360,7 +378,8 @@ __global__ void parallel_join_kernel(float* __restrict__ resid, const TA* __rest
   }
 }
 
-static int check_pick(const char* who, int E, int top, int weigh, int groups, int keep) {
+static int check_pick(const char* who, int E, int top, int weigh, int groups, int keep, const float* corr) {
+  GG_REQUIRE(!corr || (weigh == 1 && groups == 1), "%s: a correction of the choice goes with softmax scores over all experts in one group", who);
   GG_REQUIRE(weigh >= 0 && weigh <= 2, "%s: unknown way %d of weighing the chosen experts", who, weigh);
   GG_REQUIRE(groups >= 1 && keep >= 1 && keep <= groups && E % groups == 0, "%s: %d experts in %d groups of which %d are kept", who, E, groups, keep);
   GG_REQUIRE(top <= keep * (E / groups), "%s: %d choices from %d groups of %d experts", who, top, keep, E / groups);
@@ -368,13 +387,13 @@ static int check_pick(const char* who, int E, int top, int weigh, int groups, in
 }
 
 extern "C" int gg_moe_route(const void* h, const void* wr, const float* bias, int T, int D, int E, int top,
-                            int weigh, int groups, int keep, int* idx, float* wgt, float* gate, int act_dtype,
+                            int weigh, int groups, int keep, const float* corr, float scale, int* idx, float* wgt, float* gate, int act_dtype,
                             cudaStream_t stream) {
   GG_REQUIRE(T >= 0 && D > 0 && E > 0 && top > 0 && top <= E, "moe_route: bad sizes T=%d D=%d E=%d top=%d", T, D, E, top);
   GG_REQUIRE(E <= MOE_MAX_EXPERTS && top <= MOE_MAX_TOP, "moe_route: at most %d experts and %d choices a token (got %d, %d)",
              MOE_MAX_EXPERTS, MOE_MAX_TOP, E, top);
   GG_REQUIRE(h && wr && idx && wgt, "moe_route: a pointer is null");
-  if (int rc = check_pick("moe_route", E, top, weigh, groups, keep)) return rc;
+  if (int rc = check_pick("moe_route", E, top, weigh, groups, keep, corr)) return rc;
   if (T == 0) return GG_OK;
   const int tok = T > 256 ? ROUTE_TOK : 1;
   const size_t smem = (size_t)tok * D * sizeof(float);
@@ -387,7 +406,7 @@ extern "C" int gg_moe_route(const void* h, const void* wr, const float* bias, in
 #define ROUTE_LAUNCH(T_, N_)                                                                                     \
   do {                                                                                                           \
     if (smem > 28 * 1024) cudaFuncSetAttribute(moe_route_kernel<T_, N_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-    gg_launch(moe_route_kernel<T_, N_>, dim3(blocks), dim3(threads), smem, stream, (const T_*)h, (const T_*)wr, bias, T, D, E, top, weigh, groups, keep, idx, wgt, gate, vec); \
+    gg_launch(moe_route_kernel<T_, N_>, dim3(blocks), dim3(threads), smem, stream, (const T_*)h, (const T_*)wr, bias, T, D, E, top, weigh, groups, keep, corr, scale, idx, wgt, gate, vec); \
   } while (0)
   if (act_dtype == GG_F32) {
     if (tok == 1) ROUTE_LAUNCH(float, 1); else ROUTE_LAUNCH(float, ROUTE_TOK);
@@ -399,15 +418,15 @@ extern "C" int gg_moe_route(const void* h, const void* wr, const float* bias, in
 }
 
 extern "C" int gg_moe_topk(const float* z, long long z_stride, const float* bias, int T, int E, int top, int weigh, int groups, int keep,
-                           int* idx, float* wgt, cudaStream_t stream) {
+                           const float* corr, float scale, int* idx, float* wgt, cudaStream_t stream) {
   GG_REQUIRE(T >= 0 && E > 0 && top > 0 && top <= E && E <= MOE_MAX_EXPERTS && top <= MOE_MAX_TOP,
              "moe_topk: bad sizes T=%d E=%d top=%d", T, E, top);
   GG_REQUIRE(z && idx && wgt && z_stride >= E, "moe_topk: a pointer is null or the rows are too short");
-  if (int rc = check_pick("moe_topk", E, top, weigh, groups, keep)) return rc;
+  if (int rc = check_pick("moe_topk", E, top, weigh, groups, keep, corr)) return rc;
   if (T == 0) return GG_OK;
   const int warps = 4;
   gg_launch(moe_topk_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), (size_t)warps * E * sizeof(float), stream,
-            z, z_stride, bias, T, E, top, weigh, groups, keep, idx, wgt);
+            z, z_stride, bias, T, E, top, weigh, groups, keep, corr, scale, idx, wgt);
   return gg_check_launch("moe_topk");
 }
 
@@ -439,31 +458,31 @@ extern "C" int gg_moe_gather(const void* x, const int* sorted, int slots, int to
 }
 
 extern "C" int gg_moe_combine(const void* y, const int* place, const float* wgt, const void* shared_out,
-                              const float* gate, long long gate_stride, void* out, int T, int D, int top, int act_dtype, cudaStream_t stream) {
+                              const float* gate, long long gate_stride, const void* same, void* out, int T, int D, int top, int act_dtype, cudaStream_t stream) {
   GG_REQUIRE(T >= 0 && D > 0 && top > 0, "moe_combine: bad sizes T=%d D=%d top=%d", T, D, top);
   GG_REQUIRE(y && place && out && (shared_out || !gate), "moe_combine: a pointer is null");
   if (T == 0) return GG_OK;
   const int threads = D >= 1024 ? 256 : 128;
   if (act_dtype == GG_F32)
     gg_launch(moe_combine_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)y, place, wgt, (const float*)shared_out,
-              gate, gate_stride, (float*)out, D, top);
+              gate, gate_stride, (const float*)same, (float*)out, D, top);
   else if (act_dtype == GG_BF16)
     gg_launch(moe_combine_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, (const __nv_bfloat16*)y, place, wgt,
-              (const __nv_bfloat16*)shared_out, gate, gate_stride, (__nv_bfloat16*)out, D, top);
+              (const __nv_bfloat16*)shared_out, gate, gate_stride, (const __nv_bfloat16*)same, (__nv_bfloat16*)out, D, top);
   else
     return gg_fail(GG_ERR_INVALID, "moe_combine: unknown dtype %d", act_dtype);
   return gg_check_launch("moe_combine");
 }
 
 extern "C" int gg_parallel_join(float* resid, const void* mixer, const void* y, const int* place, const float* wgt, int top,
-                                const void* shared_out, const float* gate, long long gate_stride, const float* bias, float mult,
+                                const void* shared_out, const float* gate, long long gate_stride, const void* same, const float* bias, float mult,
                                 const float* norm_w, float eps, void* h, int T, int D, int act_dtype, cudaStream_t stream) {
   GG_REQUIRE(T >= 0 && D > 0 && top >= 0, "parallel_join: bad sizes T=%d D=%d top=%d", T, D, top);
   GG_REQUIRE(resid && mixer && (top == 0 || (y && place)) && (shared_out || !gate) && (h || !norm_w), "parallel_join: a pointer is null");
   const size_t smem = norm_w ? (size_t)D * sizeof(float) : 0;
   GG_REQUIRE(smem <= 200 * 1024, "parallel_join: rows of %d values do not fit in shared memory", D);
   if (T == 0) return GG_OK;
-  const size_t at = (size_t)resid | (size_t)mixer | (size_t)y | (size_t)shared_out | (size_t)bias | (size_t)norm_w | (size_t)h;
+  const size_t at = (size_t)resid | (size_t)mixer | (size_t)y | (size_t)shared_out | (size_t)same | (size_t)bias | (size_t)norm_w | (size_t)h;
   const int vec = D % 4 == 0 && at % 16 == 0;
   const int per = vec ? 4 : 1;
   int threads = ((D + per - 1) / per + 31) / 32 * 32;
@@ -472,7 +491,7 @@ extern "C" int gg_parallel_join(float* resid, const void* mixer, const void* y, 
   do {                                                                                                                           \
     if (smem > 40 * 1024) cudaFuncSetAttribute(parallel_join_kernel<T_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     gg_launch(parallel_join_kernel<T_>, dim3(T), dim3(threads), smem, stream, resid, (const T_*)mixer, (const T_*)y, place, wgt, top, \
-              (const T_*)shared_out, gate, gate_stride, bias, mult, norm_w, eps, (T_*)h, D, vec);                                 \
+              (const T_*)shared_out, gate, gate_stride, (const T_*)same, bias, mult, norm_w, eps, (T_*)h, D, vec);                                 \
   } while (0)
   if (act_dtype == GG_F32) JOIN_LAUNCH(float);
   else if (act_dtype == GG_BF16) JOIN_LAUNCH(__nv_bfloat16);

@@ -361,6 +361,16 @@ def gemm_small_m_clamped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, li
                                          ctypes.c_float(limit), ctypes.c_float(alpha), ctypes.c_float(shift), _stream()))
 
 
+def gemm_small_m_relu2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """gemm_small_m with the square of relu in its epilogue; bfloat16 out, M <= 16."""
+    M, K = x.shape
+    N = out.shape[1]
+    if w.shape != (N, K) or out.shape[0] != M or not out.is_contiguous() or out.dtype != torch.bfloat16:
+        raise KernelError("gemm_small_m_relu2: shapes do not fit")
+    _cuda(w, out)
+    _check(lib().gg_gemm_small_m_relu2(_p(x), ctypes.c_longlong(x.stride(0)), _p(w), _p(out), M, N, K, _stream()))
+
+
 _TC_STATUS = {}
 tc_launched = False       # a tcgen05 product was launched since the status word was last checked
 
@@ -390,11 +400,11 @@ def tc_ok(x: torch.Tensor, w: torch.Tensor, out_cols: int) -> bool:
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool = False,
-            pair: bool = False) -> None:
+            pair: bool = False, relu2: bool = False) -> None:
     """out[M, N] = x[M, K] @ w[N, K]^T on tcgen05 (bfloat16 in, float32 accumulate in tensor
     memory); out bfloat16 or float32.  ``gated``: w is [2N, K] (gate rows, then up rows) and
     out = silu(x Wg^T) * (x Wu^T) in bfloat16.  ``pair``: the kernel in which two CTAs on two
-    SMs share a 256 x 256 tile (cta_group::2)."""
+    SMs share a 256 x 256 tile (cta_group::2).  ``relu2`` (one CTA, bfloat16 out): the square of relu."""
     M, K = x.shape
     N = out.shape[1]
     if w.shape != ((2 * N, K) if gated else (N, K)) or out.shape[0] != M or not out.is_contiguous():
@@ -403,7 +413,9 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool = F
         raise KernelError("gemm_tc: the gated product writes bfloat16")
     if out.dtype not in (torch.float32, torch.bfloat16):
         raise KernelError("gemm_tc: out must be bfloat16 or float32")
-    mode = 2 if gated else (1 if out.dtype == torch.float32 else 0)
+    if relu2 and (gated or pair or out.dtype != torch.bfloat16):
+        raise KernelError("gemm_tc: the square of relu goes with a plain product in bfloat16 on single CTAs")
+    mode = 2 if gated else 3 if relu2 else (1 if out.dtype == torch.float32 else 0)
     global tc_launched
     tc_launched = True
     fn = lib().gg_gemm_tc2 if pair else lib().gg_gemm_tc
@@ -579,7 +591,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
                  a_group_cols: int = 0, o_group_cols: int = 0, n_padded: Optional[int] = None,
                  offsets: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None, row_div: int = 1,
                  rows: Optional[int] = None, gated: bool = False, gate: Optional[torch.Tensor] = None,
-                 gate_col0: int = 0, row_scale: Optional[torch.Tensor] = None, max_rows: int = 0) -> None:
+                 gate_col0: int = 0, row_scale: Optional[torch.Tensor] = None, max_rows: int = 0, relu2: bool = False) -> None:
     """out_g = a_g @ w_g^T for every group g (csrc/grouped_gemm.cu).  w [groups, n (2n if gated), k].
     Without ``offsets`` every group has the first ``rows`` rows of a and reads columns
     g * a_group_cols .. + k of them; with ``offsets`` [groups + 1] group g has rows offsets[g] ..
@@ -588,7 +600,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
     group g is multiplied by sigmoid(gate[a row, gate_col0 + g]).  ``row_scale`` (float32): the products
     of row r are multiplied by row_scale[row_index[r]] (row_scale[r] without a row list) before the
     activation: a factor on the input row that does not round it again.  ``max_rows``: no group has more rows
-    than this (0: not known); few rows per group run on a kernel that streams the weights once."""
+    than this (0: not known); few rows per group run on a kernel that streams the weights once.  ``relu2`` (not gated): out_g is the square of relu."""
     _cuda(w, offsets, row_index, row_scale)
     if row_scale is not None and row_scale.dtype != torch.float32:
         raise KernelError("grouped_gemm: the factors on rows are float32")
@@ -600,7 +612,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, k:
     _check(lib().gg_grouped_gemm(_p(a), ctypes.c_longlong(a.stride(0)), ctypes.c_longlong(a_group_cols), _p(row_index),
                                  int(row_div), _p(w), _p(out), ctypes.c_longlong(out.stride(0)),
                                  ctypes.c_longlong(o_group_cols), _p(offsets), M, groups, n, k,
-                                 int(n_padded if n_padded is not None else n), int(gated), _p(gate),
+                                 int(n_padded if n_padded is not None else n), 1 if gated else 2 if relu2 else 0, _p(gate),
                                  ctypes.c_longlong(gate.stride(0) if gate is not None else 0), int(gate_col0), _p(row_scale), int(max_rows),
                                  dtype_code(a.dtype), _stream()))
 
@@ -624,39 +636,44 @@ MOE_WEIGH = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2}
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], top: int,
               idx: torch.Tensor, wgt: torch.Tensor, weigh: str = "softmax_chosen", groups: int = 1, keep: int = 1,
-              gate: Optional[torch.Tensor] = None) -> None:
+              gate: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
     """Float32 logits h @ w_router^T + bias; idx [T, top] int32 = the largest, wgt [T, top]
     float32 = softmax over those ("softmax_chosen"), or the softmax over all experts divided by the
     chosen ones' sum ("softmax_all"), or each chosen logit's sigmoid as it is ("sigmoid").  ``groups`` > 1:
     only experts of the ``keep`` groups (of neighbouring experts) with the best expert can be chosen.
-    ``gate`` (float32 [T]): w_router has one row more than there are experts, whose product with h goes there."""
-    _cuda(h, w_router, bias, idx, wgt, gate)
+    ``gate`` (float32 [T]): w_router has one row more than there are experts, whose product with h goes there.
+    ``correction`` (float32, one an expert; with "softmax_all"): the choice goes by score + correction, the weights by the
+    scores alone; ``scale``: a factor on the weights."""
+    _cuda(h, w_router, bias, idx, wgt, gate, correction)
     T, D = h.shape
     E = w_router.shape[0] - (1 if gate is not None else 0)
     if gate is not None and (gate.dtype != torch.float32 or gate.numel() < T):
         raise KernelError("moe_route: the gate's logits are float32 [T]")
     if w_router.dtype != h.dtype or w_router.shape[1] != D or idx.dtype != torch.int32 or wgt.dtype != torch.float32 \
-            or (bias is not None and bias.dtype != torch.float32):
+            or any(v is not None and (v.dtype != torch.float32 or v.numel() != E) for v in (bias, correction)):
         raise KernelError("moe_route: router of the rows' dtype, bias and weights float32, choices int32")
     _check(lib().gg_moe_route(_p(h), _p(w_router), _p(bias), T, D, E, top, MOE_WEIGH[weigh], int(groups), int(keep),
-                               _p(idx), _p(wgt), _p(gate), dtype_code(h.dtype), _stream()))
+                               _p(correction), ctypes.c_float(scale), _p(idx), _p(wgt), _p(gate), dtype_code(h.dtype), _stream()))
 
 
 def moe_topk(z: torch.Tensor, bias: Optional[torch.Tensor], top: int, idx: torch.Tensor, wgt: torch.Tensor,
-             weigh: str = "softmax_chosen", groups: int = 1, keep: int = 1, experts: Optional[int] = None) -> None:
+             weigh: str = "softmax_chosen", groups: int = 1, keep: int = 1, experts: Optional[int] = None,
+             correction: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
     """moe_route's choice from logits z [T, E] (float32) that a product has already made (``experts``: only
     that many of z's columns are experts)."""
-    _cuda(z, bias, idx, wgt)
+    _cuda(z, bias, idx, wgt, correction)
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != int(experts or z.shape[1])):
+        raise KernelError("moe_topk: the correction is float32, one an expert")
     if z.dtype != torch.float32 or idx.dtype != torch.int32 or wgt.dtype != torch.float32:
         raise KernelError("moe_topk: logits and weights float32, choices int32")
     _check(lib().gg_moe_topk(_p(z), ctypes.c_longlong(z.stride(0)), _p(bias), z.shape[0], int(experts or z.shape[1]), top, MOE_WEIGH[weigh], int(groups), int(keep),
-                              _p(idx), _p(wgt), _stream()))
+                              _p(correction), ctypes.c_float(scale), _p(idx), _p(wgt), _stream()))
 
 
 def moe_align(idx: torch.Tensor, n: int, experts: int, offsets: torch.Tensor, order: torch.Tensor,
               place: torch.Tensor, pad: int = 1, tile_group: Optional[torch.Tensor] = None) -> None:
     """The n (token, choice) pairs of idx sorted by expert: offsets [experts + 1], order (pair
-    index at each place), place [n] (place of each pair).  ``pad`` > 1: every expert's places start
+    index at each place), place [n] (place of each pair; -1 where idx is no expert but past the last).  ``pad`` > 1: every expert's places start
     at a multiple of pad; order then has n + experts * (pad - 1) entries or more, -1 at places
     that hold no pair, and tile_group[i] is the expert of places pad * i .. (or -1)."""
     _cuda(idx, offsets, order, place, tile_group)
@@ -674,10 +691,10 @@ def moe_gather(x: torch.Tensor, order: torch.Tensor, top: int, out: torch.Tensor
 
 def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_group: torch.Tensor, groups: int,
                     gated: bool = False, row_entry: Optional[torch.Tensor] = None,
-                    row_scale: Optional[torch.Tensor] = None) -> None:
+                    row_scale: Optional[torch.Tensor] = None, relu2: bool = False) -> None:
     """The tcgen05 product (gemm_tc) over groups: rows 128 i .. of x belong to group tile_group[i]
     (< 0: to none, skipped) and are multiplied with that group's matrix w[g] ([groups, N, K]; gated:
-    [groups, 2N, K], out = silu(x Wg^T) * (x Wu^T)).  bfloat16; rows of x a multiple of 128.  ``row_scale``
+    [groups, 2N, K], out = silu(x Wg^T) * (x Wu^T); ``relu2``: out = the square of relu(x W^T)).  bfloat16; rows of x a multiple of 128.  ``row_scale``
     (gated, float32): the products of row r are multiplied by row_scale[row_entry[r]] before the activation."""
     global tc_launched
     M, K = x.shape
@@ -689,38 +706,40 @@ def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_gr
     if row_scale is not None and (row_scale.dtype != torch.float32 or row_entry is None or row_entry.numel() < M):
         raise KernelError("gemm_tc_grouped: float32 factors with a row list as long as x")
     tc_launched = True
-    _check(lib().gg_gemm_tc_grouped(_p(x), ctypes.c_longlong(x.stride(0)), _p(w), _p(out), M, N, K, 2 if gated else 0,
+    _check(lib().gg_gemm_tc_grouped(_p(x), ctypes.c_longlong(x.stride(0)), _p(w), _p(out), M, N, K, 2 if gated else 3 if relu2 else 0,
                                     _p(tile_group), groups, _p(row_entry), _p(row_scale), _p(tc_status(x.device)), _stream()))
 
 
 def moe_combine(y: torch.Tensor, place: torch.Tensor, wgt: Optional[torch.Tensor], shared: Optional[torch.Tensor],
-                out: torch.Tensor, top: int, gate: Optional[torch.Tensor] = None) -> None:
+                out: torch.Tensor, top: int, gate: Optional[torch.Tensor] = None,
+                same: Optional[torch.Tensor] = None) -> None:
     """out[t] = sum_j wgt[t, j] * y[place[t * top + j]] (+ shared[t]); wgt None: weights of 1; ``gate`` (float32
-    column view [T, 1] or [T]): the shared row is multiplied by sigmoid(gate[t])."""
+    column view [T, 1] or [T]): the shared row is multiplied by sigmoid(gate[t]).  ``same``: the rows that choices with a
+    place of -1 add (needed where there are such)."""
     if gate is not None and (gate.dtype != torch.float32 or gate.shape[0] != out.shape[0]):
         raise KernelError("moe_combine: the gate's logits are float32, one a token")
-    _cuda(y, place, wgt, shared, out)
+    _cuda(y, place, wgt, shared, out, same)
     T, D = out.shape
     _check(lib().gg_moe_combine(_p(y), _p(place), _p(wgt), _p(shared), _p(gate),
-                                ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _p(out), T, D, top, dtype_code(out.dtype), _stream()))
+                                ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _p(same), _p(out), T, D, top, dtype_code(out.dtype), _stream()))
 
 
 def parallel_join(resid: torch.Tensor, mixer: torch.Tensor, mult: float, bias: Optional[torch.Tensor] = None,
                   dense: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None,
                   wgt: Optional[torch.Tensor] = None, top: int = 0, gate: Optional[torch.Tensor] = None,
-                  norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, normed: Optional[torch.Tensor] = None) -> None:
+                  same: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, normed: Optional[torch.Tensor] = None) -> None:
     """resid[t] += mult * (mixer[t] + bias + sum_j wgt[t, j] * y[place[t * top + j]] + sigmoid(gate[t]) * dense[t]); every term
-    but the first is optional (wgt None: weights of 1, gate None: a factor of 1).  With ``norm_weight``: normed[t] =
+    but the first is optional (wgt None: weights of 1, gate None: a factor of 1; a place of -1 reads same[t]).  With ``norm_weight``: normed[t] =
     resid[t] / sqrt(mean(resid[t]^2) + eps) * norm_weight."""
-    _cuda(resid, mixer, bias, dense, y, place, wgt, norm_weight, normed)
+    _cuda(resid, mixer, bias, dense, y, place, wgt, same, norm_weight, normed)
     T, D = resid.shape
     if resid.dtype != torch.float32 or mixer.shape != resid.shape \
-            or any(t is not None and (t.dtype != mixer.dtype or t.shape[-1] != D) for t in (dense, y, normed)) \
+            or any(t is not None and (t.dtype != mixer.dtype or t.shape[-1] != D) for t in (dense, y, same, normed)) \
             or any(t is not None and (t.dtype != torch.float32 or t.numel() != D) for t in (bias, norm_weight)) \
             or (gate is not None and (gate.dtype != torch.float32 or gate.shape[0] != T)):
         raise KernelError("parallel_join: float32 residual, rows of its width in the activation type, float32 bias, weight and gate")
     _check(lib().gg_parallel_join(_p(resid), _p(mixer), _p(y), _p(place), _p(wgt), int(top), _p(dense), _p(gate),
-                                  ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _p(bias), ctypes.c_float(mult),
+                                  ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _p(same), _p(bias), ctypes.c_float(mult),
                                   _p(norm_weight), ctypes.c_float(eps), _p(normed), T, D, dtype_code(mixer.dtype), _stream()))
 
 
@@ -1074,6 +1093,31 @@ def qkv_norm_rope_write(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping
                                         page_size, int(interleaved), int(write_cache), _stream()))
 
 
+def qkv_row_norm_rope_write(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Optional[torch.Tensor],
+                            inv_freq: Optional[torch.Tensor], magnitude: float, q_weight: torch.Tensor, k_weight: torch.Tensor,
+                            eps: float, kcache: Optional[torch.Tensor], vcache: Optional[torch.Tensor], nh: int, nkv: int,
+                            d: int, nv: int, dv: int, page_size: int, interleaved: bool = False,
+                            write_cache: bool = True) -> None:
+    """Rows [nh*d | nkv*d | nv*dv] of qkv: the whole q part divided by its root mean square and multiplied by q_weight
+    (float32 [nh*d]), the k part by its own and k_weight [nkv*d]; then the first 2 * len(inv_freq) values of every head
+    are rotated, q in place; k and v go to the cache at slot_mapping[t] (the k part of qkv is left as it was)."""
+    _cuda(positions, slot_mapping, inv_freq, q_weight, k_weight, kcache, vcache)
+    if qkv.stride(1) != 1 or qkv.shape[1] < (nh + nkv) * d + nv * dv:
+        raise KernelError("qkv_row_norm_rope_write: rows are not contiguous or too short")
+    if inv_freq is not None and inv_freq.dtype != torch.float64:
+        raise KernelError("qkv_row_norm_rope_write: inverse frequencies must be float64")
+    for w, n in ((q_weight, nh * d), (k_weight, nkv * d)):
+        if w.dtype != torch.float32 or w.numel() != n:
+            raise KernelError("qkv_row_norm_rope_write: a norm weight is float32 of its part's width")
+    if kcache is not None and (kcache.dtype != qkv.dtype or vcache.dtype != qkv.dtype):
+        raise KernelError("qkv_row_norm_rope_write: cache and activations differ in dtype")
+    rot = 2 * inv_freq.numel() if inv_freq is not None else 0
+    _check(lib().gg_qkv_row_norm_rope_write(_p(qkv), ctypes.c_longlong(qkv.stride(0)), dtype_code(qkv.dtype), _p(positions),
+                                            _p(slot_mapping), _p(inv_freq), ctypes.c_float(magnitude), _p(q_weight), _p(k_weight),
+                                            ctypes.c_float(eps), _p(kcache), _p(vcache), qkv.shape[0], nh, nkv, d, nv, dv, rot,
+                                            page_size, int(interleaved), int(write_cache), _stream()))
+
+
 def latent_rope(src: torch.Tensor, k_col0: int, q_head: int, q_off: int, heads: int, positions: torch.Tensor,
                 inv_freq: torch.Tensor, magnitude: float, interleaved: bool, slot_mapping: Optional[torch.Tensor],
                 cache: Optional[torch.Tensor], qout: torch.Tensor, row: int, dst_col: int, write_cache: bool = True) -> None:
@@ -1232,3 +1276,74 @@ def retention_decode(proj: torch.Tensor, gate_col: int, positions: torch.Tensor,
                                      _p(positions), _p(inv_freq), _p(decay), _p(state), _p(dec_seqs), n_dec, _p(cu_q_lens),
                                      _p(context_lens), _p(state_slots), heads, d, dv, rot, int(interleaved),
                                      ctypes.c_float(kscale), ctypes.c_float(eps), _p(out), _stream()))
+
+
+# ---------------------------------------------------------------- selective scan
+SCAN_MAX_STATE = 256          # states a channel
+
+
+def scan_conv(x: torch.Tensor, conv_w: torch.Tensor, bias: Optional[torch.Tensor], conv_state: Optional[torch.Tensor],
+              cu_q_lens: torch.Tensor, context_lens: torch.Tensor, state_slots: torch.Tensor, num_seqs: int,
+              out: torch.Tensor) -> None:
+    """out = silu(short causal convolution per channel + bias) of the first C columns of x, conv_w [C, taps] float32;
+    what lies before a portion comes from conv_state [slots, taps-1, C] (float32), which is not changed."""
+    _cuda(conv_w, bias, conv_state, cu_q_lens, context_lens, state_slots, out)
+    C, taps = conv_w.shape
+    if x.stride(1) != 1 or x.shape[1] < C or out.dtype != x.dtype or tuple(out.shape) != (x.shape[0], C) or not out.is_contiguous() \
+            or any(t is not None and t.dtype != torch.float32 for t in (conv_w, bias, conv_state)):
+        raise KernelError("scan_conv: bad shapes or dtypes")
+    _check(lib().gg_scan_conv(_p(x), ctypes.c_longlong(x.stride(0)), dtype_code(x.dtype), _p(conv_w), _p(bias), _p(conv_state),
+                              _p(cu_q_lens), _p(context_lens), _p(state_slots), x.shape[0], num_seqs, C, taps, _p(out), _stream()))
+
+
+def selective_scan(x: torch.Tensor, proj: torch.Tensor, low: torch.Tensor, b_col: int, v: Optional[torch.Tensor],
+                   w_dt: Optional[torch.Tensor], dt_bias: torch.Tensor, a2: torch.Tensor, d_skip: torch.Tensor, state: torch.Tensor,
+                   conv_state: Optional[torch.Tensor], taps: int, cu_q_lens: torch.Tensor, context_lens: torch.Tensor,
+                   state_slots: torch.Tensor, num_seqs: int, single: bool, out: torch.Tensor) -> None:
+    """out = (y + d_skip x) * silu(z) with S <- exp2(dt a2) S + dt x B, y = S . C per channel, dt = softplus(v + dt_bias), from
+    and to state [slots, I, N] float32.  x [T, I] the convolution's rows, proj [T, >= 2 I] = [x before it | z], B and C columns
+    b_col .. of low.  ``single``: every sequence has one token, and with w_dt [I, rank] the step sizes' product with low's first
+    columns is made inside (v is not read).  conv_state [slots, taps-1, I] is moved on by the step's tokens."""
+    _cuda(x, w_dt, dt_bias, a2, d_skip, state, conv_state, cu_q_lens, context_lens, state_slots, out)
+    T, I = x.shape
+    N = a2.shape[1]
+    if any(t.dtype != torch.float32 for t in (dt_bias, a2, d_skip, state)) or tuple(state.shape[1:]) != (I, N) or a2.shape[0] != I \
+            or any(t is not None and (t.dtype != x.dtype or t.stride(1) != 1) for t in (proj, low, v, w_dt, out)) \
+            or tuple(out.shape) != (T, I) or dt_bias.numel() != I or d_skip.numel() != I:
+        raise KernelError("selective_scan: bad shapes or dtypes")
+    _check(lib().gg_selective_scan(_p(x), _p(proj), ctypes.c_longlong(proj.stride(0)), _p(low), ctypes.c_longlong(low.stride(0)),
+                                   int(b_col), _p(v), ctypes.c_longlong(v.stride(0) if v is not None else 0), _p(w_dt),
+                                   w_dt.shape[1] if w_dt is not None else 0, _p(dt_bias), _p(a2), _p(d_skip), _p(state),
+                                   _p(conv_state), int(taps), _p(cu_q_lens), _p(context_lens), _p(state_slots), T, num_seqs, I, N,
+                                   int(single), _p(out), dtype_code(x.dtype), _stream()))
+
+
+# ---------------------------------------------------------------- a residual of several streams
+STREAMS_MAX = 16
+
+
+def streams_join(streams: torch.Tensor, count: int, *, start: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                 w_out: Optional[torch.Tensor] = None, w_in: Optional[torch.Tensor] = None, dense: Optional[torch.Tensor] = None,
+                 y: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None, wgt: Optional[torch.Tensor] = None,
+                 top: int = 0, same: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                 normed: Optional[torch.Tensor] = None, total: Optional[torch.Tensor] = None, act_dtype=None) -> None:
+    """Between two sublayers of a residual with ``count`` streams (float32 [T, count * D]; ``start`` [T, D]: before the first one,
+    all streams are that row).  With ``w_out``: stream t <- sum_s mix[s, t] stream s + w_out[t] * r, r = dense + the experts' rows
+    (wgt, y, place, top, same as in moe_combine).  Then u = sum_s w_in[s] stream s (w_in None: the sum); normed = u /
+    sqrt(mean(u^2) + eps) * norm_weight and new streams are stored, or (no norm_weight) total = u and they are not."""
+    _cuda(streams, start, mix, w_out, w_in, dense, y, place, wgt, same, norm_weight, normed, total)
+    T, D = streams.shape[0], streams.shape[1] // count
+    if streams.dtype != torch.float32 or streams.shape[1] != count * D or not (1 <= count <= STREAMS_MAX) \
+            or any(t is not None and (t.dtype != torch.float32 or t.shape[-1] != n) for t, n in
+                   ((start, D), (mix, count), (w_out, count), (w_in, count), (norm_weight, D), (total, D))) \
+            or any(t is not None and t.shape[-1] != D for t in (dense, y, same, normed)):
+        raise KernelError("streams_join: float32 streams and weights, rows of one width")
+    rows = [t for t in (dense, y, same, normed) if t is not None]
+    dt = rows[0].dtype if rows else (act_dtype or torch.float32)
+    if any(t.dtype != dt for t in rows):
+        raise KernelError("streams_join: rows of one dtype")
+    if top and same is None:
+        same = dense if dense is not None else y         # no choice hands its input on: never read
+    _check(lib().gg_streams_join(_p(streams), _p(start), _p(dense), _p(y), _p(place), _p(wgt), int(top), _p(same), _p(mix), _p(w_out),
+                                 _p(w_in), _p(norm_weight), ctypes.c_float(eps), _p(normed), _p(total), T, count, D, dtype_code(dt),
+                                 _stream()))

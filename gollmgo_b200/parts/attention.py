@@ -121,6 +121,8 @@ class Attention:
     sink (bool: the softmax denominator has one more term exp(sink_h), a learned number a head, with no key and
     no value; tensor ``sink_name``), temperature (coef, every): the query at position p is multiplied by
     1 + coef * ln(floor((p + 1) / every) + 1),
+    row_norm (eps): before the rotation the whole q projection, all heads together, is divided by its root mean square and
+    multiplied by a weight of its width, and the k projection by its own (tensors ``row_norm_names``),
     names (local names of the q, k, v, o tensors), out_buffer (name of the workspace buffer the
     result is left in, for a mixer that runs beside another).
 
@@ -156,6 +158,9 @@ class Attention:
         if spec.get("distance_bias"):
             self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / self.nh) for h in range(self.nh)],
                                        dtype=torch.float32, device=ctx.device)
+        self.row_norm = float(spec["row_norm"]) if spec.get("row_norm") is not None else None
+        self.row_norm_names = tuple(spec.get("row_norm_names") or ("q.norm", "k.norm"))
+        self.q_norm = self.k_norm = None
         self.names = tuple(spec.get("names") or ("q_proj.weight", "k_proj.weight", "v_proj.weight", "o_proj.weight"))
         self.out_buffer = spec.get("out_buffer") or "mixer_out"
         self.nv = self.nkv // self.v_share
@@ -173,7 +178,7 @@ class Attention:
         # Steps of decoded tokens only: a bias by distance, a sink or a temperature on an attention that is plain
         # otherwise run on the decode kernel that merges inside a cluster and writes the cache itself (which takes
         # them as options; without a rotation it is given frequencies of zero).
-        plain = (self.dv == self.d and self.softcap == 0 and self.v_share == 1 and not self.bias and not self.extras
+        plain = (self.row_norm is None and self.dv == self.d and self.softcap == 0 and self.v_share == 1 and not self.bias and not self.extras
                  and self.position.rope_table() is None and not hasattr(self.position, "apply"))
         self._decode_fused = (self._mma_x and plain and FUSE_DECODE_ROPE and ctx.device.type == "cuda"
                               and self.nh // self.nkv <= 16 and ctx.page_size & (ctx.page_size - 1) == 0)
@@ -257,6 +262,9 @@ class Attention:
              o: WeightSpec((self.hidden, self.nh * self.dv))}
         if self.has_sink:
             w[self.sink_name] = WeightSpec((self.nh,), init="normal")
+        if self.row_norm is not None:
+            w[self.row_norm_names[0]] = WeightSpec((self.nh * self.d,))
+            w[self.row_norm_names[1]] = WeightSpec((self.nkv * self.d,))
         return w
 
     def load(self, get):
@@ -266,6 +274,8 @@ class Attention:
         self.w_o = get(self.names[3]).contiguous()
         if self.has_sink:
             self.sink = get(self.sink_name).float().contiguous()
+        if self.row_norm is not None:
+            self.q_norm, self.k_norm = (get(n).float().contiguous() for n in self.row_norm_names)
 
     # the optional protocol of parts/linear.py
     def takes_normed_rows(self, num_tokens):
@@ -303,6 +313,13 @@ class Attention:
                             batch.context_lens, batch.dec_seqs, n, splits,
                             part_o, part_ml, out, self.nh, self.nkv, self.d, self.ctx.page_size, window, self.scale)
 
+    def _norm_rotate_write(self, qkv, batch, kc, vc, group, writes_cache):
+        """The norms over whole projections, the rotation and the cache write."""
+        ops.qkv_row_norm_rope_write(qkv, batch.positions, batch.slot_mapping[group], self.position.rope_table(),
+                                    float(getattr(self.position, "magnitude", 1.0)), self.q_norm, self.k_norm, self.row_norm,
+                                    kc, vc, self.nh, self.nkv, self.d, self.nv, self.dv, self.ctx.page_size,
+                                    self.position.interleaved, writes_cache)
+
     def attend_general(self, x, batch, cache, writes_cache, out):
         """q, k, v projections, bias, rotation, cache write and attention on the general kernels;
         fills ``out`` [T, nh * dv] (the activation type, or float32)."""
@@ -325,9 +342,12 @@ class Attention:
                                  batch.slot_mapping[group], self._no_turn, writes_cache, sink=self.sink, slopes=self.slopes,
                                  temperature=self.temperature)
             return out
-        ops.rope_kv_write_x(qkv, batch.positions, batch.slot_mapping[group], self.position.rope_table(),
-                            float(getattr(self.position, "magnitude", 1.0)), self.qkv_bias, kc, vc, self.nh, self.nkv,
-                            self.d, self.nv, self.dv, self.ctx.page_size, self.position.interleaved, writes_cache)
+        if self.row_norm is not None:
+            self._norm_rotate_write(qkv, batch, kc, vc, group, writes_cache)
+        else:
+            ops.rope_kv_write_x(qkv, batch.positions, batch.slot_mapping[group], self.position.rope_table(),
+                                float(getattr(self.position, "magnitude", 1.0)), self.qkv_bias, kc, vc, self.nh, self.nkv,
+                                self.d, self.nv, self.dv, self.ctx.page_size, self.position.interleaved, writes_cache)
         window = int(self.window or 0)
         bt = batch.block_tables[group]
         more = dict(sink=self.sink, slopes=self.slopes, temperature=self.temperature)
@@ -369,10 +389,14 @@ class Attention:
         table = self.position.rope_table()
         flat_step = self._flat_step(batch.num_decode)
         fused = (FUSE_DECODE_ROPE and batch.num_decode > 0 and not batch.num_portions and ATTN_POLICY != "general"
-                 and not flat_step
+                 and not flat_step and self.row_norm is None
                  and not hasattr(self.position, "apply")
                  and ops.attn_decode_rope_ok(qkv.dtype, self.nh, self.nkv, self.d, table, self.position.interleaved))
-        if not fused:
+        if self.row_norm is not None:
+            if hasattr(self.position, "apply"):
+                raise TypeError("a position encoding that rewrites q and k itself cannot be used with norms over whole projections")
+            self._norm_rotate_write(qkv, batch, kc, vc, group, writes_cache)
+        elif not fused:
             ops.rope_kv_write(qkv, batch.positions, batch.slot_mapping[group], table,
                               kc, vc, self.nh, self.nkv, self.d, self.ctx.page_size,
                               self.position.interleaved, writes_cache)

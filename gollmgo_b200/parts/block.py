@@ -272,7 +272,112 @@ class SandwichBlock:
         return None
 
 
+class StreamRows:
+    """What a block of several residual streams hands to the next one: the streams hold everything, and ``rows`` is
+    the input of its first sublayer (contracted and normed)."""
+
+    def __init__(self, rows):
+        self.rows = rows
+
+
+class StreamsBlock:
+    """Instead of one residual there are ``streams`` of them, x_1 .. x_S (hyper-connections).  Sublayer q (1: the mixer,
+    2: the feed-forward) reads u = sum_s in_q[s] x_s through the layer's norm, and its result y is written back while the
+    streams are mixed: x_t <- sum_s mix_q[s, t] x_s + out_q[t] y, all at once from the old ones.  A stretch of such
+    blocks starts with S copies of the residual and ends with their sum in it, so it can stand between other blocks.
+    A layer without a feed-forward stops after the mixer.  params: streams, names (prefixes of the two sublayers'
+    tensors, with ".in", ".out" and ".mix" appended).
+
+    Everything between two sublayers is one kernel (csrc/streams.cu): the sublayer's result (of a mixture of experts
+    its rows before they are summed), the mixing, the next contraction and the next norm, so each stream is read and
+    written once per sublayer.  The streams are float32 and live in the workspace for the step."""
+
+    chains_norms = True          # forward takes next_block=
+
+    def __init__(self, layer_spec, mixer, feed_forward, mixer_norm, ffn_norm, ctx):
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.mixer_norm, self.ffn_norm = mixer_norm, ffn_norm
+        self.ctx = ctx
+        self.hidden = mixer_norm.size
+        p = layer_spec.block
+        self.streams = int(p["streams"])
+        self.names = tuple(p.get("names") or ("hc1", "hc2"))
+        if not (1 <= self.streams <= ops.STREAMS_MAX):
+            raise ValueError(f"{self.streams} residual streams are outside 1..{ops.STREAMS_MAX}")
+        if feed_forward is not None and ffn_norm is None:
+            raise ValueError("a block with a feed-forward needs the norm before it")
+        for n in (mixer_norm, ffn_norm):
+            if n is not None and not hasattr(n, "rms_weight_eps"):
+                raise TypeError(f"norm {type(n).__name__} cannot read residual streams (no rms_weight_eps)")
+        ctx.workspace.reserve("normed", ctx.max_tokens * self.hidden, ctx.act_dtype)
+        ctx.workspace.reserve("streams", ctx.max_tokens * self.streams * self.hidden, torch.float32)
+        self.w_in, self.w_out, self.mix = [None, None], [None, None], [None, None]
+
+    def _count(self):
+        return 2 if self.feed_forward is not None else 1
+
+    def weights(self):
+        w, S = {}, self.streams
+        for n in self.names[:self._count()]:
+            w.update({n + ".in": WeightSpec((S,), init="fraction"), n + ".out": WeightSpec((S,), init="fraction"),
+                      n + ".mix": WeightSpec((S, S), init="mixing")})
+        return w
+
+    def load(self, get):
+        for i, n in enumerate(self.names[:self._count()]):
+            self.w_in[i], self.w_out[i], self.mix[i] = (get(n + k).float().contiguous() for k in (".in", ".out", ".mix"))
+
+    def takes_normed_rows(self, T):
+        return False                                      # (the protocol of the pre-norm block; this one hands on StreamRows)
+
+    def follows_on(self, block):
+        """Whether this block can take its streams and first norm from ``block``."""
+        return isinstance(block, StreamsBlock) and block.streams == self.streams and block.hidden == self.hidden
+
+    def _pending(self, part, y):
+        if getattr(part, "deferred_bias", None) is not None:
+            raise ValueError("a block of several streams takes no sublayer that leaves a bias to be added")
+        return {"dense": y}
+
+    def forward(self, resid, delta, batch, cache, writes_cache=True, next_block=None):
+        T, S, ws = resid.shape[0], self.streams, self.ctx.workspace
+        x, h = ws.get("streams", T, S * self.hidden), ws.get("normed", T, self.hidden)
+        start = None                                      # the one row all streams are copies of, until they are first written
+
+        def norm_of(block, norm, i):
+            w, eps = norm.rms_weight_eps()
+            return dict(w_in=block.w_in[i], norm_weight=w, eps=eps, normed=h)
+
+        if isinstance(delta, StreamRows):
+            h = delta.rows
+        else:
+            if torch.is_tensor(delta):
+                self.mixer_norm.add_norm(resid, delta, h)            # what the block before still owes goes into the residual
+            elif delta is not None and not isinstance(delta, ResidualRows):
+                raise ValueError("a block of several streams cannot take the norm's input from the block before it")
+            start = resid
+            ops.streams_join(x, S, start=start, **norm_of(self, self.mixer_norm, 0))
+        owed, q = self._pending(self.mixer, self.mixer.forward(h, batch, cache, writes_cache)), 0
+        if self.feed_forward is not None:
+            ops.streams_join(x, S, start=start, mix=self.mix[0], w_out=self.w_out[0], **owed, **norm_of(self, self.ffn_norm, 1))
+            start, q = None, 1
+            owed = None
+            if hasattr(self.feed_forward, "forward_pending"):
+                owed = self.feed_forward.forward_pending(h, batch)
+                if owed.pop("gate") is not None:
+                    raise ValueError("a block of several streams takes no shared expert with a gate")
+            else:
+                owed = self._pending(self.feed_forward, self.feed_forward.forward(h, batch))
+        args = dict(start=start, mix=self.mix[q], w_out=self.w_out[q], **owed)
+        if next_block is not None and self.follows_on(next_block):
+            ops.streams_join(x, S, **args, **norm_of(next_block, next_block.mixer_norm, 0))
+            return StreamRows(h)
+        ops.streams_join(x, S, **args, total=resid)       # the stretch ends: the streams' sum is the residual again
+        return None
+
+
 register_block("pre_norm", PreNormBlock)
+register_block("streams", StreamsBlock)
 register_block("sandwich", SandwichBlock)
 register_block("parallel", ParallelBlock)
 register_block("post_norm", PostNormBlock)

@@ -139,8 +139,11 @@ class PlainMLP:
         T = x.shape[0]
         ws = self.ctx.workspace
         u = ws.get("ffn_up", T, self.inter)
-        linear(x, self.w_up, u)
-        ops.act(u, u, self.activation)
+        if self.activation == "relu2" and ops.small_m_ok(x, self.w_up):
+            ops.gemm_small_m_relu2(x, self.w_up, u)          # product and activation in one
+        else:
+            linear(x, self.w_up, u)
+            ops.act(u, u, self.activation)
         return linear(u, self.w_down, ws.get("ffn_out", T, self.hidden))
 
 

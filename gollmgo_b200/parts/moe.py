@@ -1,4 +1,4 @@
-"""A mixture of experts as a feed-forward: a router picks ``top`` of ``experts`` small SiLU-gated
+"""A mixture of experts as a feed-forward: a router picks ``top`` of ``experts`` small (SiLU-gated or plain)
 feed-forwards per token, their results are summed with the router's weights, and an optional
 shared expert (any registered feed-forward) runs for every token and is added.
 
@@ -19,13 +19,18 @@ g = min(gate, limit), u = clamp(up, -limit, limit) instead of silu(gate) * up;
 ``router_weigh="sigmoid"``: the weights are the sigmoids of the chosen logits, not normalised;
 ``weigh_input``: the weight multiplies the expert's input instead of its output (the first product is linear, so
 its results are multiplied in float32 before the activation and the input row is not rounded again);
+``gated=False``: an expert is down(act(up(x))) without a gate, activation "relu2" (the square of relu, in the first
+product's epilogue);
+``correction`` (with "softmax_all"): a learned number per expert is added to the scores for the choice alone;
+``router_scale``: a factor on the weights; ``identity`` = n: the router has n more outputs, experts without tensors whose
+output is their input (a choice of one costs nothing but its share of the sum);
 ``shared_gate``: the shared expert's output is multiplied by sigmoid(w . x), one number a token (the row w is
 one more row of the router's product).
 
 params: hidden_size, intermediate_size, experts, top, router_bias (bool), router_weigh, groups,
-activation, limit, alpha, shift, weigh_input, shared (a feed-forward PartSpec or None), shared_gate, names: dict
+router_scale, correction, identity, gated, activation, limit, alpha, shift, weigh_input, shared (a feed-forward PartSpec or None), shared_gate, names: dict
 with "router", "router_bias", "expert" (a format string with {e}), "gate", "up", "down", "shared" (prefix of the
-shared expert's tensors), "shared_gate".
+shared expert's tensors), "shared_gate", "correction".
 """
 from __future__ import annotations
 
@@ -48,7 +53,8 @@ TC_TILE = 128
 ROUTE_LIB_TOKENS = int(os.environ.get("GOLLMGO_B200_MOE_ROUTE_LIB_TOKENS", "512"))
 
 DEFAULT_NAMES = {"router": "router", "router_bias": "router.b", "expert": "e{e}.", "gate": "gate",
-                 "up": "up", "down": "down", "shared": "shared.", "shared_gate": "shared.sg"}
+                 "up": "up", "down": "down", "shared": "shared.", "shared_gate": "shared.sg",
+                 "correction": "correction"}
 
 
 class MixtureOfExperts:
@@ -58,9 +64,11 @@ class MixtureOfExperts:
         self.inter = int(spec["intermediate_size"])
         self.experts = int(spec["experts"])
         self.top = int(spec["top"])
-        if not (0 < self.top <= self.experts):
-            raise ValueError(f"{self.top} choices of {self.experts} experts")
-        if self.experts > ops.MOE_MAX_EXPERTS or self.top > ops.MOE_MAX_TOP:
+        self.identity = int(spec.get("identity") or 0)
+        self.choices = self.experts + self.identity            # what the router scores
+        if not (0 < self.top <= self.choices):
+            raise ValueError(f"{self.top} choices of {self.choices} experts")
+        if self.choices > ops.MOE_MAX_EXPERTS or self.top > ops.MOE_MAX_TOP:
             raise ValueError(f"the routing kernels take at most {ops.MOE_MAX_EXPERTS} experts and "
                              f"{ops.MOE_MAX_TOP} choices a token")
         self.router_bias = bool(spec.get("router_bias", True))
@@ -68,27 +76,37 @@ class MixtureOfExperts:
         if self.weigh not in ops.MOE_WEIGH:
             raise ValueError(f"router weights {self.weigh!r} are not known (known: {sorted(ops.MOE_WEIGH)})")
         self.group_count, self.group_keep = (int(g) for g in (spec.get("groups") or (1, 1)))
-        if self.experts % self.group_count or not (1 <= self.group_keep <= self.group_count) \
-                or self.top > self.group_keep * (self.experts // self.group_count):
-            raise ValueError(f"{self.experts} experts in {self.group_count} groups of which {self.group_keep} are kept "
+        if self.choices % self.group_count or not (1 <= self.group_keep <= self.group_count) \
+                or self.top > self.group_keep * (self.choices // self.group_count):
+            raise ValueError(f"{self.choices} experts in {self.group_count} groups of which {self.group_keep} are kept "
                              f"do not give {self.top} choices")
-        self.activation = spec.get("activation") or "silu"
-        if self.activation not in ("silu", "clamped_swish"):
-            raise ValueError(f"activation {self.activation!r} is not supported (known: silu, clamped_swish)")
+        self.correction = bool(spec.get("correction", False))
+        self.router_scale = float(spec.get("router_scale", 1.0))
+        if self.correction and (self.weigh != "softmax_all" or self.group_count > 1):
+            raise ValueError("a correction of the choice goes with softmax scores over all experts in one group")
+        if self.identity and self.group_count > 1:
+            raise ValueError("groups of experts and experts that hand on their input do not go together")
+        self.gated = bool(spec.get("gated", True))
+        self.activation = spec.get("activation") or ("silu" if self.gated else "relu2")
+        known = ("silu", "clamped_swish") if self.gated else ("relu2",)
+        if self.activation not in known:
+            raise ValueError(f"activation {self.activation!r} is not supported (known: {', '.join(known)})")
         if self.activation == "clamped_swish":
             self.limit = float(spec["limit"])
             self.alpha = float(spec.get("alpha", 1.702))
             self.shift = float(spec.get("shift", 1.0))
         self.weigh_input = bool(spec.get("weigh_input", False))
-        if self.weigh_input and self.activation != "silu":
-            raise ValueError("weights on the experts' input go with the silu-gated experts")
+        if self.weigh_input and (self.activation != "silu" or self.identity):
+            raise ValueError("weights on the experts' input go with the silu-gated experts alone")
         self.names = {**DEFAULT_NAMES, **(spec.get("names") or {})}
         shared = spec.get("shared")
         self.shared = build_feed_forward(shared, ctx) if shared is not None else None
         self.shared_gate = bool(spec.get("shared_gate", False)) and self.shared is not None
         # the router's rows: one per expert, then the shared expert's gate, then (for a product whose rows
         # start on 16-byte borders) rows of zeros
-        self.router_rows = -(-(self.experts + 1) // 8) * 8 if self.shared_gate else self.experts
+        self.router_rows = self.choices + (1 if self.shared_gate else 0)
+        if self.shared_gate or self.identity:
+            self.router_rows = -(-self.router_rows // 8) * 8
         ws, T = ctx.workspace, ctx.max_tokens
         n = T * self.top
         self.tc_ok = (ctx.act_dtype == torch.bfloat16 and GEMM_POLICY != "lib" and self.hidden % 8 == 0
@@ -104,11 +122,11 @@ class MixtureOfExperts:
         ws.reserve("moe_tiles", slots // TC_TILE + 1, torch.int32)
         ws.reserve("moe_in", slots * self.hidden, ctx.act_dtype)
         ws.reserve("moe_act", slots * self.inter, ctx.act_dtype)
-        if self.activation != "silu":
+        if self.activation == "clamped_swish":
             ws.reserve("moe_gate_up", slots * 2 * self.inter, ctx.act_dtype)
         ws.reserve("moe_rows", slots * self.hidden, ctx.act_dtype)
         ws.reserve("moe_out", T * self.hidden, ctx.act_dtype)
-        self.w_router = self.b_router = self.w_gate_up = self.w_down = None
+        self.w_router = self.b_router = self.w_gate_up = self.w_down = self.choice_correction = None
 
     def _slots(self, n):
         """Places of the padded row block: every expert's rows rounded up to whole tiles."""
@@ -118,11 +136,14 @@ class MixtureOfExperts:
         return self.names["expert"].format(e=e) + self.names[which]
 
     def weights(self):
-        m = {self.names["router"]: WeightSpec((self.experts, self.hidden))}
+        m = {self.names["router"]: WeightSpec((self.choices, self.hidden))}
         if self.router_bias:
-            m[self.names["router_bias"]] = WeightSpec((self.experts,))
+            m[self.names["router_bias"]] = WeightSpec((self.choices,))
+        if self.correction:
+            m[self.names["correction"]] = WeightSpec((self.choices,), init="normal")
         for e in range(self.experts):
-            m[self._expert(e, "gate")] = WeightSpec((self.inter, self.hidden))
+            if self.gated:
+                m[self._expert(e, "gate")] = WeightSpec((self.inter, self.hidden))
             m[self._expert(e, "up")] = WeightSpec((self.inter, self.hidden))
             m[self._expert(e, "down")] = WeightSpec((self.hidden, self.inter))
         if self.shared is not None:
@@ -133,15 +154,19 @@ class MixtureOfExperts:
 
     def load(self, get):
         self.w_router = get(self.names["router"]).contiguous()
-        if self.shared_gate:
-            w, sg = self.w_router, get(self.names["shared_gate"])
-            dt = torch.float32 if torch.float32 in (w.dtype, sg.dtype) else w.dtype
+        if self.router_rows != self.choices:
+            w = self.w_router
+            sg = get(self.names["shared_gate"]) if self.shared_gate else None
+            dt = torch.float32 if sg is not None and torch.float32 in (w.dtype, sg.dtype) else w.dtype
             self.w_router = torch.zeros(self.router_rows, self.hidden, dtype=dt, device=w.device)
-            self.w_router[:self.experts] = w.to(dt)
-            self.w_router[self.experts:self.experts + 1] = sg.to(dt)
+            self.w_router[:self.choices] = w.to(dt)
+            if sg is not None:
+                self.w_router[self.choices:self.choices + 1] = sg.to(dt)
+        self.choice_correction = get(self.names["correction"]).float().contiguous() if self.correction else None
         self.b_router = get(self.names["router_bias"]).to(torch.float32).contiguous() if self.router_bias else None
-        # [experts, 2 * inter, hidden]: an expert's gate rows, then its up rows
-        self.w_gate_up = torch.stack([torch.cat([get(self._expert(e, "gate")), get(self._expert(e, "up"))], dim=0)
+        # [experts, 2 * inter, hidden]: an expert's gate rows, then its up rows (its up rows alone without a gate)
+        first = ("gate", "up") if self.gated else ("up",)
+        self.w_gate_up = torch.stack([torch.cat([get(self._expert(e, k)) for k in first], dim=0)
                                       for e in range(self.experts)]).contiguous()
         self.w_down = torch.stack([get(self._expert(e, "down")) for e in range(self.experts)]).contiguous()
         if self.shared is not None:
@@ -153,21 +178,22 @@ class MixtureOfExperts:
 
     def _route(self, x):
         """route(x), and the logits of the shared expert's gate [T, 1] (None without one)."""
-        T, ws, E = x.shape[0], self.ctx.workspace, self.experts
+        T, ws, E = x.shape[0], self.ctx.workspace, self.choices
+        more = dict(correction=self.choice_correction, scale=self.router_scale)
         idx, wgt = ws.get("moe_idx", T, self.top), ws.get("moe_wgt", T, self.top)
         gate = None
         if T >= ROUTE_LIB_TOKENS and x.dtype == torch.bfloat16:
             # a long step: the logits are a product like any other (bfloat16 rows, float32 sums and result)
             z = ws.get("moe_logits", T, self.router_rows)
             linear(x, self.w_router, z)
-            ops.moe_topk(z, self.b_router, self.top, idx, wgt, self.weigh, self.group_count, self.group_keep, experts=E)
+            ops.moe_topk(z, self.b_router, self.top, idx, wgt, self.weigh, self.group_count, self.group_keep, experts=E, **more)
             if self.shared_gate:
                 gate = z[:, E:E + 1]
         else:
-            w = self.w_router
+            w = self.w_router[:E]
             if self.shared_gate:
-                gate, w = ws.get("moe_shared_gate", T, 1), w[:E + 1]
-            ops.moe_route(x, w, self.b_router, self.top, idx, wgt, self.weigh, self.group_count, self.group_keep, gate=gate)
+                gate, w = ws.get("moe_shared_gate", T, 1), self.w_router[:E + 1]
+            ops.moe_route(x, w, self.b_router, self.top, idx, wgt, self.weigh, self.group_count, self.group_keep, gate=gate, **more)
         return idx, wgt, gate
 
     def _activate(self, gate_up, a):
@@ -176,7 +202,7 @@ class MixtureOfExperts:
     def forward(self, x, batch):
         p = self.forward_pending(x, batch)
         out = self.ctx.workspace.get("moe_out", x.shape[0], self.hidden)
-        ops.moe_combine(p["y"], p["place"], p["wgt"], p["dense"], out, p["top"], gate=p["gate"])
+        ops.moe_combine(p["y"], p["place"], p["wgt"], p["dense"], out, p["top"], gate=p["gate"], same=p["same"])
         return out
 
     def forward_pending(self, x, batch):
@@ -185,6 +211,7 @@ class MixtureOfExperts:
         T, ws = x.shape[0], self.ctx.workspace
         n, E = T * self.top, self.experts
         idx, wgt, sgate = self._route(x)
+        relu2 = not self.gated
         on_input = wgt if self.weigh_input else None
         place = ws.get("moe_place", 1, n)
         offsets = ws.get("moe_offsets", 1, E + 1)
@@ -196,8 +223,9 @@ class MixtureOfExperts:
             xin = ws.get("moe_in", slots, self.hidden)
             ops.moe_gather(x, order, self.top, xin)
             a = ws.get("moe_act", slots, self.inter)
-            if self.activation == "silu":
-                ops.gemm_tc_grouped(xin, self.w_gate_up, a, tiles, E, gated=True, row_entry=order, row_scale=on_input)
+            if self.activation != "clamped_swish":
+                ops.gemm_tc_grouped(xin, self.w_gate_up, a, tiles, E, gated=self.gated, row_entry=order, row_scale=on_input,
+                                    relu2=relu2)
             else:
                 gu = ws.get("moe_gate_up", slots, 2 * self.inter)
                 ops.gemm_tc_grouped(xin, self.w_gate_up, gu, tiles, E)
@@ -208,9 +236,9 @@ class MixtureOfExperts:
             order = ws.get("moe_order", 1, n)
             ops.moe_align(idx, n, E, offsets, order, place)
             a = ws.get("moe_act", n, self.inter)
-            if self.activation == "silu":
+            if self.activation != "clamped_swish":
                 ops.grouped_gemm(x, self.w_gate_up, a, self.inter, self.hidden, E, offsets=offsets, row_index=order,
-                                 row_div=self.top, rows=n, gated=True, row_scale=on_input, max_rows=T)
+                                 row_div=self.top, rows=n, gated=self.gated, row_scale=on_input, max_rows=T, relu2=relu2)
             else:
                 gu = ws.get("moe_gate_up", n, 2 * self.inter)
                 ops.grouped_gemm(x, self.w_gate_up, gu, 2 * self.inter, self.hidden, E, offsets=offsets, row_index=order,
@@ -219,7 +247,8 @@ class MixtureOfExperts:
             y = ws.get("moe_rows", n, self.hidden)
             ops.grouped_gemm(a, self.w_down, y, self.hidden, self.inter, E, offsets=offsets, rows=n, max_rows=T)
         shared = self.shared.forward(x, batch) if self.shared is not None else None
-        return {"y": y, "place": place, "wgt": None if self.weigh_input else wgt, "top": self.top, "dense": shared, "gate": sgate}
+        return {"y": y, "place": place, "wgt": None if self.weigh_input else wgt, "top": self.top, "dense": shared, "gate": sgate,
+                "same": x if self.identity else None}
 
 
 register_feed_forward("moe", MixtureOfExperts)

@@ -59,6 +59,15 @@ class RunEntry:
     mix_input: bool = False
 
 
+def looped_run_order(num_layers: int, start: int = 0, stop: int = 0, times: int = 1, mix_input: bool = False) -> Tuple[RunEntry, ...]:
+    """The layers in the order they run: those from ``start`` to before ``stop`` ``times`` times in a row, every pass
+    with cache entries of its own; ``mix_input``: the embedding output is mixed in before the first layer of each pass."""
+    runs = [(i, False) for i in range(start)]
+    runs += [(i, mix_input and i == start) for _ in range(times) for i in range(start, stop)]
+    runs += [(i, False) for i in range(max(start, stop), num_layers)]
+    return tuple(RunEntry(i, cache, mix_input=mix) for cache, (i, mix) in enumerate(runs))
+
+
 @dataclass(frozen=True)
 class ModelSpec:
     architecture: str

@@ -36,6 +36,10 @@ def random_tensor(name: str, spec: WeightSpec, seed: int, device, dtype: torch.d
         t = torch.empty(spec.shape, dtype=torch.float32, device=device)
         t.uniform_(0.2, 0.8, generator=gen)
         return t.to(dtype)
+    if spec.init == "mixing":                     # a square mixing matrix: near the identity
+        t = torch.empty(spec.shape, dtype=torch.float32, device=device)
+        t.normal_(0.0, 0.1, generator=gen)
+        return (t + torch.eye(spec.shape[0], device=device)).to(dtype)
     if len(spec.shape) <= 1 and spec.init != "normal":      # a norm's weight (a vector, or one number)
         t = (torch.zeros if spec.init == "offset" else torch.ones)(spec.shape, dtype=torch.float32, device=device)
         if norm_jitter:
