@@ -165,12 +165,17 @@ def reference_arm(args) -> int:
 # Rimidra: the Fapudra shape of equal width, heads, kv heads, head size, window, experts, vocabulary and number of
 # layers, with as many recurrent layers of equal state size (it has the parallel blocks, the windowed attention with
 # a bias by distance and the mixtures of experts; a Rimidra token also runs the shared expert).
+# Matusun: the Fapudra shape of equal width, heads, kv heads, head size, window, number of experts, choices, vocabulary and
+# layer runs, with as many recurrent layers of equal inner width (it has a state-space mixer, a windowed attention and
+# the mixtures of experts; Matusun's experts have two matrices instead of three and are half as wide again, a token also
+# runs the shared expert).
 DESIGN_PAIRS = {
     "tekenex": [("tekenex_w2048", "llama_mqa_w2048"), ("tekenex_w4096", "llama_mqa_w4096")],
     "bevuvik": [("bevuvik_w2048", "llama_gqa_w2048"), ("bevuvik_w4096", "llama_gqa_w4096")],
     "fapudra": [("fapudra_w2048", "bevuvik_w2048"), ("fapudra_w4096", "bevuvik_w4096")],
     "fivesun": [("fivesun_w2048", "bevuvik_w2048"), ("fivesun_w4096", "bevuvik_w4096")],
     "rimidra": [("rimidra_w2048", "fapudra_w2048"), ("rimidra_w4096", "fapudra_w4096")],
+    "matusun": [("matusun_w2048", "fapudra_w2048"), ("matusun_w4096", "fapudra_w4096")],
 }
 
 

@@ -30,7 +30,7 @@ from .registry import register_mixer
 _NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "x": "x", "dt": "dt", "dt_bias": "dt.b", "A_log": "A_log",
           "D": "D", "o": "o"}
 # Steps of at most this many single tokens make the step sizes inside the recurrence (every token reads W_dt again).
-FUSE_DT_TOKENS = int(os.environ.get("GOLLMGO_B200_SCAN_FUSE_DT", "16"))
+FUSE_DT_TOKENS = int(os.environ.get("GOLLMGO_B200_SCAN_FUSE_DT", "8"))
 
 
 def _up8(n):
